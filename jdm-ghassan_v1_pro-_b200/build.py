@@ -34,6 +34,11 @@ NVCC_FLAGS = [
     "--use_fast_math", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
     "-Xptxas", "-v", "-DNDEBUG",
 ]
+# Kernels of layer-list models keep IEEE division, square roots and math functions: their fp32 mode is meant to be exact.
+PRECISE_PREFIX = "layers_"
+# Sources behind one kind of model, for a process that serves nothing else and finds no library (`ensure_layers`).
+LAYERS_PART = ("layers_", "gemm_")
+LAYERS_SO = os.path.join(HERE, "_gb200_layers.so")
 CXX_FLAGS = ["-O2", "-std=c++20", "-fPIC", "-fvisibility=hidden", "-Wall", "-Wno-unused-function",
              "-pthread"]
 
@@ -139,25 +144,47 @@ def build_host_sanitized(kind: str, verbose=False) -> str:
     return target
 
 
-def build_cuda(verbose=False, force=False):
+def _nvcc_flags(src):
+    if os.path.basename(src).startswith(PRECISE_PREFIX):
+        return [f for f in NVCC_FLAGS if f != "--use_fast_math"]
+    return NVCC_FLAGS
+
+
+def build_cuda(verbose=False, force=False, part=None, target=None):
+    """Compile the device library; ``part``: only the sources whose names start with one of these prefixes, linked to
+    ``target``."""
     os.makedirs(os.path.join(BUILD, "cuda"), exist_ok=True)
-    srcs = _sources("cuda", ".cu")
+    srcs = [s for s in _sources("cuda", ".cu") if part is None or os.path.basename(s).startswith(part)]
     hdrs = _headers("cuda")
+    target = target or CUDA_SO
     jobs = []
     objs = []
     for s in srcs:
         o = os.path.join(BUILD, "cuda", os.path.basename(s) + ".o")
         objs.append(o)
         if force or _newer([s] + hdrs, o):
-            jobs.append(([NVCC] + NVCC_FLAGS + ["-I" + os.path.join(CSRC, "cuda"), "-c", s, "-o", o],
+            jobs.append(([NVCC] + _nvcc_flags(s) + ["-I" + os.path.join(CSRC, "cuda"), "-c", s, "-o", o],
                          o + ".log"))
     with cf.ThreadPoolExecutor(max_workers=os.cpu_count() or 4) as ex:
         for out in ex.map(lambda j: _run(*j), jobs):
             if verbose and out.strip():
                 print(out)
-    if jobs or not os.path.exists(CUDA_SO):
-        _link([NVCC, "-shared"], CUDA_SO, objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-lcudart"])
-    return CUDA_SO
+    if jobs or _newer(objs, target):
+        _link([NVCC, "-shared"], target, objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-lcudart"])
+    return target
+
+
+def ensure_layers() -> str:
+    """Device library for a process that only serves layer-list models: the full one when it is there and up to date,
+    else a library of just the sources they need (compiled on the first call)."""
+    import fcntl
+    srcs = [s for s in _sources("cuda", ".cu") if os.path.basename(s).startswith(LAYERS_PART)] + _headers("cuda")
+    if not _newer(srcs, CUDA_SO):
+        return CUDA_SO
+    os.makedirs(BUILD, exist_ok=True)
+    with open(os.path.join(BUILD, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build_cuda(part=LAYERS_PART, target=LAYERS_SO)
 
 
 def build_all(verbose=False, force=False):

@@ -13,8 +13,9 @@
     python -m ghassan_b200.cli.infer devices
     python -m ghassan_b200.cli.infer logits    --model model.gguf --prompt "salam" [--out logits.f32]
 
-GGUF is the deploy format (weights + tokenizer + configuration in one file); legacy .gai files and training
-checkpoints load too.  Generation options: --temp --top-k --top-p --min-p --repeat --no-repeat-ngram --max-tokens
+GGUF is the deploy format (weights + tokenizer + configuration in one file); legacy .gai files, training checkpoints and
+folders with config.json and safetensors (models/registry.py) load too.  Without a tokenizer, `generate` and `logits` take
+token ids: --ids "12 7 99".  Generation options: --temp --top-k --top-p --min-p --repeat --no-repeat-ngram --max-tokens
 --seed --greedy --system --persona darija|en --no-adaptive --no-stream --retrieve-index <path> --retrieve-direct.
 """
 from __future__ import annotations
@@ -35,7 +36,7 @@ def _parser() -> argparse.ArgumentParser:
     ap.add_argument("command", choices=["chat", "generate", "info", "quantize", "bench", "tokenize", "export", "eval",
                                         "perplexity", "devices", "logits"])
     for name in ("model", "prompt", "out", "profile", "tokenizer", "text", "checkpoint", "suite", "shards", "prefix", "system",
-                 "persona", "retrieve-index", "categories", "format", "compat"):
+                 "persona", "retrieve-index", "categories", "format", "compat", "ids"):
         ap.add_argument("--" + name)
     for name, typ in (("temp", float), ("top-k", int), ("top-p", float), ("min-p", float), ("repeat", float),
                       ("no-repeat-ngram", int), ("max-tokens", int), ("seed", int), ("tokens", int), ("prompt-tokens", int),
@@ -98,12 +99,18 @@ def _sampling(a):
     return sp
 
 
+def _ids(text: str) -> List[int]:
+    return [int(t) for t in text.replace(",", " ").split()]
+
+
 def _load(a, batch=1, ctx=0):
     from ..inference import model_io as IO
     from ..inference.generator import Generator
     if not a.model:
         raise SystemExit("--model is required")
     m = IO.load_model(a.model, a.tokenizer or "")
+    if (a.rope_scale is not None or a.yarn_mscale is not None) and not hasattr(m.cfg, "rope_scale"):
+        raise SystemExit("--rope-scale and --yarn-mscale do not apply to %s models" % m.cfg.architecture)
     if a.rope_scale is not None or a.yarn_mscale is not None:      # run-time context extension (perplexity sweeps)
         if a.rope_scale is not None:
             m.cfg.rope_scale = float(a.rope_scale)
@@ -206,6 +213,12 @@ def main(argv: Optional[List[str]] = None) -> int:
         return 0
     m, gen = _load(a, ctx=a.ctx or 0)
     sp = _sampling(a)
+    if cmd == "generate" and a.ids:
+        res = gen.generate([_ids(a.ids)], max_new_tokens=a.max_tokens or 256, sampling=sp, stop_tokens=None if gen.tok is not None else ())
+        print(" ".join(map(str, res.tokens[0])))
+        if a.stats:
+            print("  [prefill %.0f ms | decode %.1f tok/s | %s]" % (res.prefill_seconds * 1e3, res.decode_tokens_per_second, res.stopped[0]))
+        return 0
     if cmd == "generate":
         if gen.tok is None:
             raise SystemExit("model has no tokenizer; pass --tokenizer")
@@ -248,7 +261,7 @@ def main(argv: Optional[List[str]] = None) -> int:
         ChatSession(gen, o).run_repl()
         return 0
     if cmd == "logits":
-        ids = gen.encode_prompt(a.prompt or "", add_bos=True)
+        ids = _ids(a.ids) if a.ids else gen.encode_prompt(a.prompt or "", add_bos=True)
         import torch
         if hasattr(gen.engine, "all_logits"):
             # the reference's report (tools/inference_cli.cpp:748-812 there): every position's logits to --out as
@@ -288,8 +301,9 @@ def main(argv: Optional[List[str]] = None) -> int:
             r = E.perplexity_shards(gen, a.shards, a.prefix or "val", max_tokens=batches * bs * seq_len, window=seq_len)
         else:
             raise SystemExit("perplexity requires --text or --shards")
-        print("  rope_scale  : %.3f" % m.cfg.rope_scale)
-        print("  yarn_mscale : %.3f" % m.cfg.rope_mscale())
+        if hasattr(m.cfg, "rope_scale"):
+            print("  rope_scale  : %.3f" % m.cfg.rope_scale)
+            print("  yarn_mscale : %.3f" % m.cfg.rope_mscale())
         print("  mean_nll    : %.8f" % r["nll"])
         print("  perplexity  : %.6f" % r["perplexity"])
         print("  tokens      : %d" % r["tokens"])

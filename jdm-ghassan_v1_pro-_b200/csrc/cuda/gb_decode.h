@@ -19,7 +19,8 @@ enum {
   GB_W_GGML_Q8_0 = 2,  // 32 values: f16 scale + 32 x i8                       (34 B)   GGUF type 8
   GB_W_Q4_0 = 3,       // 32 values: f16 scale + 16 B, byte i = code[2i+1]<<4 | code[2i], v = (code-8)*s   (18 B)
   GB_W_Q8_64 = 4,      // 64 values: f32 scale + 64 x i8                       (68 B)   internal Q8_0
-  GB_W_Q4_1 = 5        // 32 values: f16 scale, f16 min + 16 B, v = code*s + min (20 B)
+  GB_W_Q4_1 = 5,       // 32 values: f16 scale, f16 min + 16 B, v = code*s + min (20 B)
+  GB_W_F32 = 6         // 4 B / value (layer-list models in true fp32 only)
 };
 long long gb_wfmt_row_bytes(int fmt, int K);   // -1 when K does not fit the block size
 

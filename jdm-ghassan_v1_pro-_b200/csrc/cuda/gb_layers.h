@@ -1,0 +1,113 @@
+// Kernels of models described layer by layer (attention with a kept-prefix window, sink, output gate; Mamba-2; dense
+// feed-forward; norms on the sublayers' outputs).  Every kernel works on `B` sequences of `n` consecutive new tokens
+// (row r = b * n + t) that continue from the per-sequence state in `st` (position of the first new token: abs_pos),
+// so a prompt, a portion of one and a single decoded token are the same call.  Sizes are run-time values; rows of
+// weights and activations that feed a matrix product are padded with zeros to a multiple of eight elements.
+//
+// dtype: element type of weights, activations and attention cache: 1 = bf16, 2 = fp32.  What belongs to the state (SSM
+// states, positions), norms, scores, gates of the recurrence and the residual is fp32 for either.
+#pragma once
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "gb_decode.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+// x[r, :] = table[ids[r], :] in fp32 (pitch d) and in the compute type (pitch ld16; the columns past d are zeroed).
+int gb_ll_embed(const int* ids, const void* table, long long ld_table, int vocab, float* x, void* x16, long long ld16, int rows,
+                int d, int dtype, cudaStream_t st);
+// x_out = x + (y / rms(y)) * w, x16 = compute-type copy of x_out.  x16 may be NULL; x_out may be x.
+int gb_ll_postnorm(const float* y, long long ldy, const float* x, const float* w, float eps, float* x_out, void* x16,
+                   long long ld16, int rows, int d, int dtype, cudaStream_t st);
+// out[r, :] = compute-type copy of (x / rms(x)) * w for x row `row_idx[r]` (NULL: row r).
+int gb_ll_norm_rows(const float* x, const int* row_idx, const float* w, float eps, void* out, long long ldo, int rows, int d,
+                    int dtype, cudaStream_t st);
+// v = cap * tanh(v / cap) in place over [rows, n] fp32.
+int gb_ll_softcap(float* v, long long ld, int rows, int n, float cap, cudaStream_t st);
+// C[M, N] = A[M, K] B[N, K]^T in fp32 (true fp32 products); K a multiple of 4, rows 16-byte aligned.
+int gb_ll_gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N, int K,
+                   cudaStream_t st);
+// act[r, j] = silu(g) * u for gate/up columns interleaved in blocks of 64 (g0..g63, u0..u63, g64..), fp32.
+int gb_ll_swiglu_f32(const float* gu, long long ld, float* act, long long lda, int rows, int E, cudaStream_t st);
+// st[b].abs_pos += n (and the cache_len the sampler's transcript shares), pos_out[b] = new position.
+int gb_ll_advance(gb_seq_state* state, int* pos_out, int B, int n, cudaStream_t st);
+
+// ------------------------------------------------------------------------------------------------ token-step GEMV
+// out[b, j] = W[j, :] . v_b for B <= 8 sequences, where v_b is made by a prologue inside the kernel:
+//   prologue 0: v = x16 (compute type, pitch ldx)
+//   prologue 1: x_new = x + norm(y) * w1 (y NULL: x_new = x), written to x_out by one block; v = x_new, or
+//               norm(x_new) * w2 when w2 is given
+//   prologue 2: v = norm_parts(y16 * silu(z16)) * w1, `parts` equal parts each by its own root mean square
+// swiglu != 0: W holds gate/up rows interleaved in blocks of 64 (N = 2 E rows) and out[b, j] = silu(gate_j) * up_j.
+// softcap > 0: out = cap * tanh(out / cap).
+typedef struct gb_ll_gemv_args {
+  const void* W; int fmt, N, K;          // K: stored row length (values beyond `d` are zero)
+  int B, dtype, prologue, swiglu;
+  int d;                                 // true length of v
+  const void* x16; long long ldx;
+  const float* x; const float* y; long long ldy; const float* w1; const float* w2; float eps; float* x_out;
+  const void* y16; long long ldy16; const void* z16; long long ldz; int parts;
+  void* out; long long ldo; int out_f32; float softcap;
+} gb_ll_gemv_args;
+int gb_ll_gemv(const gb_ll_gemv_args* a, cudaStream_t st);
+
+// ------------------------------------------------------------------------------------------------ attention
+// Cache rows of a sequence: positions below `keep` have row = position for good; later positions share a ring,
+// row = keep + (position - keep) % (cap - keep).  Key j is visible to query i iff j <= i and (window == 0 or
+// i - j < window or j < keep).  The ring must hold window - 1 + n positions (all of them when window == 0).
+typedef struct gb_ll_attn_args {
+  int dtype, B, n;
+  int H, G;                              // query heads, key/value heads
+  int dk, dv, dkp, dvp;                  // head sizes and their padded row lengths in q and the caches (padding is zero)
+  int rot_dims, rot_half;                // rotated leading dimensions; 0: pairs (2i, 2i+1), 1: pairs (i, i + rot_dims/2)
+  const double* freq;                    // [rot_dims / 2] angular frequencies
+  int qk_norm;                           // divide q and k by their root mean square after the rotation
+  float eps, scale;
+  int window, keep, cap;
+  const void* proj; long long ld_proj;   // [rows, q: H*dk | k: G*dk | v: G*dv | gate: H*dv (gate != 0)]
+  int gate;                              // multiply the heads' outputs by sigmoid(gate columns)
+  const float* sink;                     // [H] or NULL: exp(sink) joins the soft-max denominator
+  void* q;                               // [rows, H, dkp]
+  void* cache_k; void* cache_v;          // [B, cap, G, dkp] / [B, cap, G, dvp]
+  void* out; long long ldo;              // [rows, H*dv]
+  float* scratch; int splits;            // token step: B * H * splits * (dvp + 2) floats
+  const gb_seq_state* st;
+  int pos0_max;                          // host's upper bound of abs_pos over the B sequences (tile counts); -1 unknown
+  int* status;
+} gb_ll_attn_args;
+int gb_ll_qkv_store(const gb_ll_attn_args* a, cudaStream_t st);     // rotation, norm, q out, k and v into the cache
+int gb_ll_attn_prefill(const gb_ll_attn_args* a, cudaStream_t st);  // any dtype and head size up to 256
+int gb_ll_attn_tc_ok(const gb_ll_attn_args* a);                     // 0 when the tensor-core kernel covers the shapes
+int gb_ll_attn_tc(const gb_ll_attn_args* a, cudaStream_t st);       // bf16
+int gb_ll_attn_decode(const gb_ll_attn_args* a, cudaStream_t st);   // n == 1
+
+// ------------------------------------------------------------------------------------------------ Mamba-2
+typedef struct gb_ll_mamba_args {
+  int dtype, B, n;
+  int H, P, N, G, taps;                  // heads, head size, state size, groups, convolution taps
+  int Pp, Np;                            // padded row lengths of xh and bc / cc
+  int Ns;                                // row length of a stored state (N rounded up to 4)
+  const void* proj; long long ld_proj;   // [rows, z: H*P | x: H*P | B: G*N | C: G*N | dt: H]
+  const float* conv_w; const float* conv_b;   // [channels, taps], [channels] for channels x | B | C
+  const float* dt_bias; const float* A_log; const float* D;
+  const float* norm_w; int norm_groups; float eps;
+  void* conv_state;                      // [B, taps, channels]: input of position p in row p % taps
+  float* ssm;                            // [B, H, P, Ns]
+  void* xh; void* bc; void* cc;          // convolved: [rows, H, Pp], [rows, G, Np], [rows, G, Np]
+  void* y; long long ld_y;               // [rows, H*P]
+  void* out; long long ld_out;           // [rows, H*P] gated and normed
+  const gb_seq_state* st;
+  float* chunk_ws;                       // chunked scan: see gb_ll_ssd_ws_floats
+  int* status;
+} gb_ll_mamba_args;
+int gb_ll_conv(const gb_ll_mamba_args* a, cudaStream_t st);
+int gb_ll_scan(const gb_ll_mamba_args* a, cudaStream_t st);         // recurrence token by token, any dtype
+int gb_ll_gated_norm(const gb_ll_mamba_args* a, cudaStream_t st);
+int gb_ll_mamba_step(const gb_ll_mamba_args* a, cudaStream_t st);   // n == 1: convolution + recurrence in one kernel
+
+#ifdef __cplusplus
+}
+#endif

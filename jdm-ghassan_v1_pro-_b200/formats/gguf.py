@@ -18,6 +18,7 @@ from typing import Dict, List, Optional, Sequence
 import numpy as np
 
 from .. import _gb200_host as H
+from .loaded import LoadedModel  # noqa: F401  (re-exported)
 from ..data.tokenizer import N_SPECIAL, UNK, Tokenizer
 from ..models.config import ModelConfig
 
@@ -243,17 +244,6 @@ def export_gguf(path: str, cfg: ModelConfig, named: Dict[str, np.ndarray], token
                 w.add_tensor("layers.%d.moe_bias" % l, b, GGML_F32)
     w.write(path)
     return {"path": path, "profile": prof.name, "tensors": w.tensor_count, "metadata": w.metadata_count, "weight_bytes": total}
-
-
-@dataclass
-class LoadedModel:
-    cfg: ModelConfig
-    named: Dict[str, np.ndarray]          # fp32 tensors by parameter name
-    moe_bias: List[np.ndarray]
-    tokenizer: Optional[Tokenizer]
-    metadata: dict
-    tensor_types: Dict[str, int]
-    raw: Optional["H.GgufFile"] = None
 
 
 def _meta_str(md, key, default=""):

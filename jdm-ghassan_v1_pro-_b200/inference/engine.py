@@ -18,18 +18,17 @@ from __future__ import annotations
 import os
 
 import ctypes
-from dataclasses import dataclass
 from typing import Dict, List, Optional, Sequence
 
 import numpy as np
 import torch
 
-from .. import _gb200_host as H
 from ..models.config import ModelConfig
 from ..models.cuda_model import CudaModel
 from ..ops import decode as D
 from ..ops import kernels as K
 from ..utils import canary as CA
+from .token_loop import SamplingParams, TokenLoop  # noqa: F401  (SamplingParams is re-exported)
 
 PINNED_TOKENS = 8
 
@@ -39,39 +38,11 @@ def _lib_status(dev):
     return _lib.status_word(dev)
 
 
-@dataclass
-class SamplingParams:
-    temperature: float = 0.8
-    top_k: int = 40
-    top_p: float = 0.92
-    min_p: float = 0.05
-    repetition_penalty: float = 1.12
-    repetition_window: int = 128
-    frequency_penalty: float = 0.0
-    presence_penalty: float = 0.0
-    no_repeat_ngram: int = 0
-    greedy: bool = False
-    seed: int = 0
-
-    def to_native(self) -> "H.SamplingConfig":
-        c = H.SamplingConfig()
-        for k, v in self.__dict__.items():
-            setattr(c, k, v)
-        c.validate()
-        return c
-
-    def device_ok(self) -> bool:
-        """Settings the device sampler takes; anything else is sampled on the host from the logits."""
-        if self.no_repeat_ngram > 0 or self.repetition_window > 1024:
-            return False
-        return self.greedy or self.temperature <= 0 or 1 <= self.top_k <= 1024
-
-
 class _Layer:
     pass
 
 
-class InferenceEngine:
+class InferenceEngine(TokenLoop):
     """Weights in decode formats + KV cache + one captured decode step for ``batch`` sequences."""
 
     def __init__(self, cfg: ModelConfig, named: Dict[str, np.ndarray], fmt: str = "f16", batch: int = 1,
@@ -161,10 +132,8 @@ class InferenceEngine:
         self.weight_bytes = sum(w.nbytes for L in self.layers for w in (L.wqkv, L.wo, L.wg, L.wu, L.wd)) + self.head.nbytes
         # ---- decode state and buffers (all static: one graph serves every step)
         B = batch
-        self.state = CA.zeros(B, D.STATE_INTS, **i32)
+        self._init_loop(B, V, max_len)
         self.slot_pos = CA.zeros(B, max_len, **i32)
-        self.pos = CA.zeros(B, **i32)
-        self.cur_tok = CA.zeros(B, **i32)
         self.x = [CA.zeros(B, d, **f32) for _ in range(2)]
         self.x_mid = CA.zeros(B, d, **f32)
         self.xb = CA.zeros(B, d, **c16)
@@ -179,23 +148,12 @@ class InferenceEngine:
         self.r_w = CA.zeros(B, max(1, cfg.moe_top_k), **f32)
         self.dense_idx = CA.zeros(B, 1, **i32)          # dense FFN = one "expert" with weight 1
         self.dense_w = torch.ones(B, 1, **f32)
-        self.logits = CA.zeros(B, V, **f32)
         # split-KV: enough (sequence, kv head, split) blocks to cover the GPU; a warp walks its slots one by one,
         # so at batch 1 the cache is cut fine (a few slots per warp) and the partial results merged afterwards
         self.splits = int(min(64, max(8, 512 // (B * cfg.num_kv_heads))))
         self.att_scratch = CA.zeros(B * cfg.num_heads * self.splits * (cfg.head_dim + 2), **f32)
         self.att_ticket = CA.zeros(B * cfg.num_kv_heads, **i32)
         self.cos_sin = K.rope_table(torch.from_numpy(cfg.rope_inv_freq()), max(cfg.max_seq_len, max_len) + 1, self.dev)
-        self.hist_cap = max_len + 8
-        self.history = CA.zeros(B, self.hist_cap, **i32)
-        self.hist_len = CA.zeros(B, **i32)
-        self.uniforms = CA.zeros(max_len, B, **f32)      # one row of draws per sampling step
-        self.tok_log = CA.zeros(B, max_len, **i32)
-        self.step = CA.zeros(1, **i32)
-        self.stop = CA.zeros(8, **i32)
-        self.n_stop = 0
-        self.graph: Optional[torch.cuda.CUDAGraph] = None
-        self._graph_key = None
         self.mega: Optional[D.MegaArgs] = None
         if single_kernel is None:
             single_kernel = os.environ.get("GB200_DECODE_MEGA", "1") != "0"
@@ -204,9 +162,6 @@ class InferenceEngine:
         self.prefill_chunk = min(prefill_chunk, max_len)
         self._prefill_model: Optional[CudaModel] = None
         self._named = named
-        self.rng = H.Rng(1)
-        self._uni_host = torch.zeros(max_len, B, dtype=torch.float32).pin_memory()
-        self._host_step = 0
 
     # ------------------------------------------------------------------ single-kernel step
     def _build_mega(self):
@@ -320,19 +275,6 @@ class InferenceEngine:
             D.expert_swiglu(L.wg, L.wu, 0, self.E, d, self.xb, self.dense_idx, 1, False, self.act)
             D.expert_down(L.wd, 0, d, self.E, self.act, self.dense_idx, self.dense_w, 1, False, self.x_mid, x_out)
 
-    def _sample_args(self, sp: SamplingParams) -> D.SampleArgs:
-        a = D.SampleArgs()
-        a.logits, a.ld, a.B, a.V = self.logits.data_ptr(), self.logits.stride(0), self.B, self.cfg.vocab_size
-        n = sp.to_native()
-        a.temperature, a.top_k, a.top_p, a.min_p = n.temperature, n.top_k, n.top_p, n.min_p
-        a.rep_penalty, a.freq_penalty, a.presence_penalty = n.repetition_penalty, n.frequency_penalty, n.presence_penalty
-        a.rep_window, a.greedy = n.repetition_window, int(n.greedy)
-        a.history, a.hist_cap, a.hist_len = self.history.data_ptr(), self.hist_cap, self.hist_len.data_ptr()
-        a.uniforms, a.out_tok, a.state = self.uniforms.data_ptr(), self.cur_tok.data_ptr(), self.state.data_ptr()
-        a.stop, a.n_stop = self.stop.data_ptr(), self.n_stop
-        a.tok_log, a.log_cap, a.step = self.tok_log.data_ptr(), self.tok_log.shape[1], self.step.data_ptr()
-        return a
-
     def _forward_token(self):
         """Embedding of ``cur_tok`` through all layers to fp32 logits; advances the per-sequence state."""
         cfg = self.cfg
@@ -359,60 +301,7 @@ class InferenceEngine:
             D.gemv(self.head, self.xb, self.logits)
         D.decode_advance(self.state, self.pos, self.cap, PINNED_TOKENS)
 
-    def _step_eager(self, sp: Optional[SamplingParams]):
-        self._forward_token()
-        if sp is not None:
-            D.sample(self._sample_args(sp))
-
-    def decode_steps(self, n: int, sp: SamplingParams, use_graph: bool = True):
-        """Run ``n`` decode steps (forward of ``cur_tok`` + sampling of the next token) without host reads."""
-        if not sp.device_ok():
-            raise ValueError("these sampling settings need the host sampler: use Generator.generate")
-        key = (sp.temperature, sp.top_k, sp.top_p, sp.min_p, sp.repetition_penalty, sp.repetition_window,
-               sp.frequency_penalty, sp.presence_penalty, sp.greedy, self.n_stop)
-        self._draw_uniforms(n)
-        if use_graph and (self.graph is None or self._graph_key != key):
-            self._step_eager(sp)          # a real step, run eagerly: first-use set-up must happen outside capture
-            n -= 1
-            torch.cuda.synchronize()
-            g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g, capture_error_mode="thread_local"):   # other threads (prefetch, checkpoint writer) may call CUDA
-                self._step_eager(sp)
-            self.graph, self._graph_key = g, key
-        for _ in range(max(0, n)):
-            if use_graph:
-                self.graph.replay()
-            else:
-                self._step_eager(sp)
-
-    def _draw_uniforms(self, n: int):
-        """Draws for the next ``n`` sampling steps: rows [done, done + n) of the device table the sampler indexes with
-        its own step counter.  Each row is written once per generation, so the asynchronous copy never races with
-        the host filling later rows."""
-        lo = self._host_step
-        hi = min(lo + n, self._uni_host.shape[0])
-        for s in range(lo, hi):
-            for b in range(self.B):
-                self._uni_host[s, b] = self.rng.uniform()
-        if hi > lo:
-            self.uniforms[lo:hi].copy_(self._uni_host[lo:hi], non_blocking=True)
-        self._host_step = lo + n
-
     # ------------------------------------------------------------------ prompt
-    def reset(self, seed: int = 0):
-        self.state.zero_()
-        self.pos.zero_()
-        self.hist_len.zero_()
-        self.step.zero_()
-        self._host_step = 0
-        self.rng.reseed(seed if seed else 1)
-
-    def set_stop_tokens(self, ids: Sequence[int]):
-        ids = list(ids)[:8]
-        self.n_stop = len(ids)
-        if ids:
-            self.stop[:len(ids)].copy_(torch.tensor(ids, dtype=torch.int32))
-
     def _prefill_net(self) -> CudaModel:
         if self._prefill_model is None:
             m = CudaModel(self.cfg, self.B, self.prefill_chunk, self.dt, self.dev, ce_chunks=1, use_segments=False, train=False)
@@ -464,11 +353,3 @@ class InferenceEngine:
             self.cur_tok.copy_(prompts[:, j])
             self._forward_token()
         # logits of the last prompt token are in self.logits; cur_tok is set by the first sample call
-
-    def sample_first(self, sp: SamplingParams):
-        self._draw_uniforms(1)
-        D.sample(self._sample_args(sp))
-
-    def transcript(self, n_new: int) -> torch.Tensor:
-        """Tokens sampled so far, [B, n_new] on the host (one device->host copy)."""
-        return self.tok_log[:, :n_new].cpu()

@@ -77,6 +77,9 @@ class Generator:
         eng.reset(sp.seed)
         eng.set_stop_tokens(sorted(stop_ids))
         max_new = min(max_new_tokens, eng.tok_log.shape[1])
+        limit = getattr(eng, "token_limit", None)             # an engine whose caches bound the length of a sequence
+        if limit is not None:
+            max_new = min(max_new, limit - n + 1)
         t0 = time.perf_counter()
         host_only = getattr(eng, "host_only", False)          # the CPU engine: host sampler, no device to wait for
         eng.prefill(torch.from_numpy(np.stack(ids)).to(torch.int32))

@@ -1,0 +1,298 @@
+"""Configuration of models described layer by layer.
+
+A ``config.json`` of this kind names its architecture and lists the layers; each entry has the type of its mixer, the
+mixer's sizes and constants, and its feed-forward (or none).  A mixer type is one class in :data:`MIXERS` that reads its
+entry, checks it and says which tensors it owns; the engine has the matching kernels.  Another design that is a list of
+such layers is another entry in ``models/registry.py``.
+"""
+from __future__ import annotations
+
+import json
+import math
+from dataclasses import dataclass, field
+from typing import Dict, List, Optional, Tuple
+
+import numpy as np
+
+from ..utils.log import log_warn
+
+
+def _need(cond, msg):
+    if not cond:
+        raise ValueError(msg)
+
+
+def _int(d, key, lo=1, hi=2 ** 31 - 1, default=None):
+    v = d.get(key, default)
+    _need(isinstance(v, int) and not isinstance(v, bool) and lo <= v <= hi, f"'{key}' must be an integer in [{lo}, {hi}], got {v!r}")
+    return v
+
+
+def _num(d, key, positive=True, default=None):
+    v = d.get(key, default)
+    _need(isinstance(v, (int, float)) and not isinstance(v, bool) and math.isfinite(v) and (v > 0 or not positive),
+          f"'{key}' must be a {'positive ' if positive else ''}number, got {v!r}")
+    return float(v)
+
+
+@dataclass(frozen=True)
+class RotaryScaling:
+    """Wavelength-dependent slow-down of the rotation: long wavelengths by ``factor``, short ones not at all."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
+class Rotary:
+    dims: int                       # leading dimensions of a head that turn
+    base: float
+    half: bool = False              # pairs (i, i + dims/2) instead of (2i, 2i + 1)
+    scaling: Optional[RotaryScaling] = None
+
+    def frequencies(self) -> np.ndarray:
+        """Angular frequency per pair, float64 [dims / 2]."""
+        i = np.arange(self.dims // 2, dtype=np.float64)
+        f = np.power(float(self.base), -2.0 * i / max(1, self.dims))
+        s = self.scaling
+        if s is None:
+            return f
+        turns = s.original * f / (2.0 * math.pi)                 # full turns within the original context
+        ramp = (turns - s.low) / (s.high - s.low) if s.high != s.low else np.zeros_like(f)
+        mixed = (1.0 - ramp) * f / s.factor + ramp * f
+        return np.where(turns > s.high, f, np.where(turns < s.low, f / s.factor, mixed))
+
+    @classmethod
+    def parse(cls, d: Optional[dict]) -> Optional["Rotary"]:
+        if not d:
+            return None
+        sc = d.get("scaling")
+        dims = _int(d, "dims", 0)
+        _need(dims % 2 == 0, "'rot.dims' must be even")
+        return cls(dims, _num(d, "base"), False,
+                   None if not sc else RotaryScaling(_num(sc, "factor"), _num(sc, "low"), _num(sc, "high"), _num(sc, "original")))
+
+
+@dataclass(frozen=True)
+class AttentionMixer:
+    """Grouped-query attention: rotary positions, an optional weightless RMS norm of q and k, a sliding window that keeps the
+    first tokens, a soft-max sink per head, a sigmoid gate on the heads' outputs."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: Optional[Rotary] = None
+    window: int = 0                 # 0: every earlier token is visible
+    keep_first: int = 0
+    qk_norm: bool = True
+    sink: bool = True
+    gate: bool = True
+    kind = "attention"
+
+    @classmethod
+    def parse(cls, d: dict) -> "AttentionMixer":
+        mask = d.get("mask") or {}
+        m = cls(_int(d, "heads"), _int(d, "kv_heads"), _int(d, "dim", 1, 256), _int(d, "vdim", 1, 256), _num(d, "scale", False),
+                Rotary.parse(d.get("rot")), _int(mask, "size", 1) if mask.get("size") is not None else 0,
+                _int(mask, "keep_first", 0, default=0))
+        _need(m.heads % m.kv_heads == 0, "'heads' must be a multiple of 'kv_heads'")
+        _need(m.rot is None or m.rot.dims <= m.dim, "'rot.dims' exceeds 'dim'")
+        return m
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.vdim
+
+    def projection_rows(self) -> List[Tuple[str, int]]:
+        """Tensors that read the mixer's input, in the order in which their rows are stacked."""
+        rows = [("q", self.heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)]
+        return rows + ([("g", self.heads * self.vdim)] if self.gate else [])
+
+    def tensors(self, width: int) -> Dict[str, tuple]:
+        t = {n: (r, width) for n, r in self.projection_rows()}
+        if self.sink:
+            t["sink"] = (self.heads,)
+        t["o"] = (width, self.out_features)
+        return t
+
+
+@dataclass(frozen=True)
+class Mamba2Mixer:
+    """State-space mixer with a scalar decay per head, a short causal convolution and a gated norm in equal groups."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_groups: int
+    kind = "mamba2"
+
+    @classmethod
+    def parse(cls, d: dict) -> "Mamba2Mixer":
+        m = cls(_int(d, "heads"), _int(d, "vdim"), _int(d, "state", 1, 256), _int(d, "groups"), _int(d, "conv", 1, 32),
+                _int(d, "norm_groups", default=1))
+        _need(m.heads % m.groups == 0, "'heads' must be a multiple of 'groups'")
+        _need(m.out_features % m.norm_groups == 0, "'norm_groups' must divide heads * vdim")
+        return m
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        return self.out_features + 2 * self.groups * self.state
+
+    def projection_rows(self) -> List[Tuple[str, int]]:
+        return [("in", self.out_features + self.channels + self.heads)]
+
+    def tensors(self, width: int) -> Dict[str, tuple]:
+        t = {n: (r, width) for n, r in self.projection_rows()}
+        t.update({"conv": (self.channels, self.conv), "conv.b": (self.channels,), "dt_bias": (self.heads,), "A_log": (self.heads,),
+                  "D": (self.heads,), "norm": (self.out_features,), "o": (width, self.out_features)})
+        return t
+
+
+MIXERS = {c.kind: c for c in (AttentionMixer, Mamba2Mixer)}
+
+
+@dataclass(frozen=True)
+class DenseMlp:
+    ff: int
+    kind = "dense"
+
+    @classmethod
+    def parse(cls, d: Optional[dict]) -> Optional["DenseMlp"]:
+        if d is None:
+            return None
+        _need(d.get("kind", "dense") == "dense", f"unknown feed-forward kind {d.get('kind')!r}")
+        return cls(_int(d, "ff"))
+
+    def tensors(self, width: int) -> Dict[str, tuple]:
+        return {"gate": (self.ff, width), "up": (self.ff, width), "down": (width, self.ff)}
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: object
+    mlp: Optional[DenseMlp]
+    weights: int                    # index of the layer whose tensors this one uses (itself, unless shared)
+
+
+@dataclass
+class LayerListConfig:
+    architecture: str
+    vocab_size: int
+    hidden_size: int
+    eps: float
+    layers: List[LayerSpec]
+    logit_softcap: float = 0.0
+    max_seq_len: int = 65536        # positions are computed, not tabulated: a serving default, not a limit of the model
+    extra: dict = field(default_factory=dict)
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @classmethod
+    def from_json(cls, d: dict) -> "LayerListConfig":
+        raw = d.get("layers")
+        _need(isinstance(raw, list) and raw, "'layers' must be a non-empty list")
+        specs: List[LayerSpec] = []
+        for i, e in enumerate(raw):
+            try:
+                kind = e.get("type")
+                _need(kind in MIXERS, f"unknown layer type {kind!r} (known: {', '.join(sorted(MIXERS))})")
+                own, seen = i, {i}
+                while raw[own].get("weights_of") is not None:
+                    own = raw[own]["weights_of"]
+                    _need(isinstance(own, int) and 0 <= own < len(raw) and own not in seen, "'weights_of' does not lead to a layer with tensors")
+                    seen.add(own)
+                spec = LayerSpec(MIXERS[kind].parse(e.get("mixer") or {}), DenseMlp.parse(e.get("mlp")), own)
+            except ValueError as err:
+                raise ValueError(f"layer {i}: {err}") from None
+            specs.append(spec)
+        for i, s in enumerate(specs):
+            if s.weights != i:
+                o = specs[s.weights]
+                a, b = ({k: v for k, v in m.tensors(1).items()} for m in (s.mixer, o.mixer))
+                _need(type(s.mixer) is type(o.mixer) and a == b and s.mlp == o.mlp,
+                      f"layer {i}: shares the tensors of layer {s.weights} but has other sizes")
+        cap = d.get("logit_softcap")
+        return cls(str(d.get("architecture", "")), _int(d, "vocab"), _int(d, "width"), _num(d.get("norm") or {}, "eps"), specs,
+                   0.0 if cap is None else _num(d, "logit_softcap"))
+
+    @classmethod
+    def from_file(cls, path: str) -> "LayerListConfig":
+        with open(path, "r", encoding="utf-8") as f:
+            return cls.from_json(json.load(f))
+
+    def tensor_shapes(self) -> Dict[str, tuple]:
+        """Every tensor of the model by its name in the file."""
+        d = self.hidden_size
+        out = {"embed": (self.vocab_size, d)}
+        for i, s in enumerate(self.layers):
+            if s.weights != i:
+                continue
+            p = f"l{i}."
+            out[p + "norm1"] = (d,)
+            if s.mlp is not None:
+                out[p + "norm2"] = (d,)
+            out.update({p + "mix." + n: sh for n, sh in s.mixer.tensors(d).items()})
+            if s.mlp is not None:
+                out.update({p + "mlp." + n: sh for n, sh in s.mlp.tensors(d).items()})
+        out["final.norm"] = (d,)
+        out["head"] = (self.vocab_size, d)
+        return out
+
+    def count_parameters(self) -> int:
+        return sum(int(np.prod(s)) for s in self.tensor_shapes().values())
+
+    def summary(self) -> str:
+        kinds: Dict[str, int] = {}
+        for s in self.layers:
+            kinds[s.mixer.kind] = kinds.get(s.mixer.kind, 0) + 1
+        shared = sum(1 for i, s in enumerate(self.layers) if s.weights != i)
+        return (f"{self.architecture} vocab={self.vocab_size} d={self.hidden_size} L={self.num_layers} ("
+                + ", ".join(f"{n} {k}" for k, n in sorted(kinds.items())) + (f", {shared} with shared tensors" if shared else "") + ")"
+                + (f" softcap={self.logit_softcap:g}" if self.logit_softcap > 0 else ""))
+
+
+def check_tensors(cfg: LayerListConfig, named) -> None:
+    """Raise when a tensor is missing or has another shape; name what belongs to no layer."""
+    want = cfg.tensor_shapes()
+    for n, shape in want.items():
+        _need(n in named, f"missing tensor '{n}'")
+        _need(tuple(named[n].shape) == tuple(shape), f"tensor '{n}' has shape {tuple(named[n].shape)}, expected {tuple(shape)}")
+    extra = sorted(set(named) - set(want))
+    if extra:
+        log_warn("[model] %d tensors belong to no layer and are not used (first: '%s')" % (len(extra), extra[0]))
+
+
+def random_parameters(cfg: LayerListConfig, seed: int = 0, dtype=None, device="cpu"):
+    """Random tensors of the right shapes and sane scales (benchmarks and demonstrations): matrices ~ N(0, 1/in), norms
+    around one, decays between slow and fast."""
+    import torch
+    g = torch.Generator(device="cpu").manual_seed(seed)
+    dtype = dtype or torch.bfloat16
+    out = {}
+    for n, shape in cfg.tensor_shapes().items():
+        leaf = n.split(".")[-1] if not n.endswith("conv.b") else "conv.b"
+        if leaf in ("norm1", "norm2", "norm"):
+            t = 1.0 + 0.1 * torch.randn(shape, generator=g)
+        elif leaf == "A_log":
+            t = torch.log(torch.empty(shape).uniform_(0.5, 8.0, generator=g))
+        elif leaf == "dt_bias":
+            t = torch.empty(shape).uniform_(-5.0, -1.0, generator=g)
+        elif leaf in ("D", "sink"):
+            t = torch.randn(shape, generator=g)
+        elif leaf == "conv.b":
+            t = 0.1 * torch.randn(shape, generator=g)
+        elif leaf == "embed":
+            t = torch.randn(shape, generator=g)
+        else:
+            t = torch.randn(shape, generator=g) * shape[-1] ** -0.5
+        out[n] = t.to(dtype).to(device)
+    return out

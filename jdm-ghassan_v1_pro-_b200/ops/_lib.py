@@ -46,6 +46,14 @@ def available() -> bool:
     return os.path.exists(_SO)
 
 
+def use(path: str) -> None:
+    """Take the kernels from another library file (before the first launch)."""
+    global _SO
+    if _lib is not None and path != _SO:
+        raise RuntimeError("a kernel library is loaded already")
+    _SO = path
+
+
 def lib():
     """Load (once) and return the kernel library."""
     global _lib

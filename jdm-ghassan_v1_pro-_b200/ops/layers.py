@@ -1,0 +1,133 @@
+"""Launchers for the kernels of layer-list models (``csrc/cuda/layers_*.cu``; contract in ``gb_layers.h``)."""
+from __future__ import annotations
+
+import ctypes
+
+import torch
+
+from . import _lib
+
+c_int, c_ll, c_vp, c_float = ctypes.c_int, ctypes.c_longlong, ctypes.c_void_p, ctypes.c_float
+
+DTYPE = {torch.bfloat16: 1, torch.float32: 2}
+W_FMT = {torch.bfloat16: 1, torch.float32: 6}        # stored-row formats of the GEMV kernels
+GEMV_MAX_BATCH = 8
+GEMV_MAX_SMEM = 200 * 1024
+FINAL_NORM_MAX = 4096                                # widest row whose last norm the GEMV prologue takes along
+
+
+class GemvArgs(ctypes.Structure):
+    _fields_ = [
+        ("W", c_vp), ("fmt", c_int), ("N", c_int), ("K", c_int),
+        ("B", c_int), ("dtype", c_int), ("prologue", c_int), ("swiglu", c_int), ("d", c_int),
+        ("x16", c_vp), ("ldx", c_ll),
+        ("x", c_vp), ("y", c_vp), ("ldy", c_ll), ("w1", c_vp), ("w2", c_vp), ("eps", c_float), ("x_out", c_vp),
+        ("y16", c_vp), ("ldy16", c_ll), ("z16", c_vp), ("ldz", c_ll), ("parts", c_int),
+        ("out", c_vp), ("ldo", c_ll), ("out_f32", c_int), ("softcap", c_float),
+    ]
+
+
+class AttnArgs(ctypes.Structure):
+    _fields_ = [
+        ("dtype", c_int), ("B", c_int), ("n", c_int), ("H", c_int), ("G", c_int),
+        ("dk", c_int), ("dv", c_int), ("dkp", c_int), ("dvp", c_int),
+        ("rot_dims", c_int), ("rot_half", c_int), ("freq", c_vp), ("qk_norm", c_int), ("eps", c_float), ("scale", c_float),
+        ("window", c_int), ("keep", c_int), ("cap", c_int),
+        ("proj", c_vp), ("ld_proj", c_ll), ("gate", c_int), ("sink", c_vp),
+        ("q", c_vp), ("cache_k", c_vp), ("cache_v", c_vp), ("out", c_vp), ("ldo", c_ll),
+        ("scratch", c_vp), ("splits", c_int), ("st", c_vp), ("pos0_max", c_int), ("status", c_vp),
+    ]
+
+
+class MambaArgs(ctypes.Structure):
+    _fields_ = [
+        ("dtype", c_int), ("B", c_int), ("n", c_int),
+        ("H", c_int), ("P", c_int), ("N", c_int), ("G", c_int), ("taps", c_int), ("Pp", c_int), ("Np", c_int), ("Ns", c_int),
+        ("proj", c_vp), ("ld_proj", c_ll),
+        ("conv_w", c_vp), ("conv_b", c_vp), ("dt_bias", c_vp), ("A_log", c_vp), ("D", c_vp),
+        ("norm_w", c_vp), ("norm_groups", c_int), ("eps", c_float),
+        ("conv_state", c_vp), ("ssm", c_vp), ("xh", c_vp), ("bc", c_vp), ("cc", c_vp),
+        ("y", c_vp), ("ld_y", c_ll), ("out", c_vp), ("ld_out", c_ll), ("st", c_vp), ("chunk_ws", c_vp), ("status", c_vp),
+    ]
+
+
+def _p(t):
+    return None if t is None else c_vp(t.data_ptr())
+
+
+def _call(name, *args):
+    _lib.check_rc(getattr(_lib.lib(), name)(*args, _lib.stream_ptr()), name)
+
+
+def embed(ids, table, x, x16, d):
+    _call("gb_ll_embed", _p(ids), _p(table), c_ll(table.stride(0)), c_int(table.shape[0]), _p(x), _p(x16), c_ll(x16.stride(0)),
+          c_int(ids.numel()), c_int(d), c_int(DTYPE[x16.dtype]))
+
+
+def postnorm(y, x, w, eps, x_out, x16, rows, d):
+    """``x_out = x + y / rms(y) * w`` and its compute-type copy ``x16``."""
+    _call("gb_ll_postnorm", _p(y), c_ll(y.stride(0)), _p(x), _p(w), c_float(eps), _p(x_out), _p(x16), c_ll(x16.stride(0)),
+          c_int(rows), c_int(d), c_int(DTYPE[x16.dtype]))
+
+
+def norm_rows(x, row_idx, w, eps, out, rows, d):
+    _call("gb_ll_norm_rows", _p(x), _p(row_idx), _p(w), c_float(eps), _p(out), c_ll(out.stride(0)), c_int(rows), c_int(d),
+          c_int(DTYPE[out.dtype]))
+
+
+def softcap(v, rows, n, cap):
+    _call("gb_ll_softcap", _p(v), c_ll(v.stride(0)), c_int(rows), c_int(n), c_float(cap))
+
+
+def gemm_f32(a, b, out, rows):
+    """``out[:rows] = a[:rows] @ b^T`` with fp32 products (no reduced-precision mode)."""
+    _call("gb_ll_gemm_f32", _p(a), c_ll(a.stride(0)), _p(b), c_ll(b.stride(0)), _p(out), c_ll(out.stride(0)), c_int(rows),
+          c_int(b.shape[0]), c_int(b.shape[1]))
+
+
+def swiglu_f32(gu, act, rows, E):
+    _call("gb_ll_swiglu_f32", _p(gu), c_ll(gu.stride(0)), _p(act), c_ll(act.stride(0)), c_int(rows), c_int(E))
+
+
+def advance(state, pos_out, n):
+    _call("gb_ll_advance", _p(state), _p(pos_out), c_int(state.shape[0]), c_int(n))
+
+
+def gemv(a: GemvArgs):
+    _call("gb_ll_gemv", ctypes.byref(a))
+
+
+def qkv_store(a: AttnArgs):
+    _call("gb_ll_qkv_store", ctypes.byref(a))
+
+
+def attn_prefill(a: AttnArgs):
+    _call("gb_ll_attn_prefill", ctypes.byref(a))
+
+
+def attn_tc_ok(a: AttnArgs) -> bool:
+    return hasattr(_lib.lib(), 'gb_ll_attn_tc_ok') and _lib.lib().gb_ll_attn_tc_ok(ctypes.byref(a)) == 0
+
+
+def attn_tc(a: AttnArgs):
+    _call("gb_ll_attn_tc", ctypes.byref(a))
+
+
+def attn_decode(a: AttnArgs):
+    _call("gb_ll_attn_decode", ctypes.byref(a))
+
+
+def conv(a: MambaArgs):
+    _call("gb_ll_conv", ctypes.byref(a))
+
+
+def scan(a: MambaArgs):
+    _call("gb_ll_scan", ctypes.byref(a))
+
+
+def mamba_step(a: MambaArgs):
+    _call("gb_ll_mamba_step", ctypes.byref(a))
+
+
+def gated_norm(a: MambaArgs):
+    _call("gb_ll_gated_norm", ctypes.byref(a))

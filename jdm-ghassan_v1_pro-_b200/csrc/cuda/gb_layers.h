@@ -100,11 +100,16 @@ typedef struct gb_ll_mamba_args {
   void* y; long long ld_y;               // [rows, H*P]
   void* out; long long ld_out;           // [rows, H*P] gated and normed
   const gb_seq_state* st;
-  float* chunk_ws;                       // chunked scan: see gb_ll_ssd_ws_floats
+  float* chunk_ws;                       // chunked scan: gb_ll_ssd_ws_floats floats, or NULL (no cutting into segments)
   int* status;
 } gb_ll_mamba_args;
 int gb_ll_conv(const gb_ll_mamba_args* a, cudaStream_t st);
 int gb_ll_scan(const gb_ll_mamba_args* a, cudaStream_t st);         // recurrence token by token, any dtype
+// The recurrence in chunks of 128 tokens on the tensor cores: bf16, P <= 128, N <= 128, Pp 64 or 128, Np 128.  `segments`:
+// runs that a sequence is cut into, 0 = by the number of SMs.
+int gb_ll_ssd_ok(const gb_ll_mamba_args* a);                        // 0 when the shapes are covered
+long long gb_ll_ssd_ws_floats(int B, int H, int P, int Ns, int n, int segments);
+int gb_ll_ssd(const gb_ll_mamba_args* a, int segments, cudaStream_t st);
 int gb_ll_gated_norm(const gb_ll_mamba_args* a, cudaStream_t st);
 int gb_ll_mamba_step(const gb_ll_mamba_args* a, cudaStream_t st);   // n == 1: convolution + recurrence in one kernel
 

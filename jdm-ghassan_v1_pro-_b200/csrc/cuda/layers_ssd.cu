@@ -1,0 +1,538 @@
+// Mamba-2 state recurrence over many tokens on the tensor cores (contract in gb_layers.h): chunks of 128 tokens, the
+// state of a head resident in tensor memory from chunk to chunk.
+//
+// With L_t the running sum of the log decays inside a chunk (fp32), the chunk's outputs and its new state are
+//   y_t = sum_{s <= t} (C_t . B_s) exp(L_t - L_s) dt_s x_s  +  exp(L_t) C_t . S_prev  +  D x_t
+//   S   = exp(L_last) S_prev + sum_s exp(L_last - L_s) dt_s B_s x_s^T
+// (the block form of the recurrence: T. Dao, A. Gu, "Transformers are SSMs", 2024).  x, B and C are bf16 as the
+// convolution leaves them.  Everything else is fp32; where an fp32 quantity has to be an operand (the weights of the
+// first sum, the scaled x of the state update, S_prev itself) it enters as two bf16 terms, value and remainder, so that
+// products keep 16 bits of it, and the state accumulates in fp32.
+//
+// One CTA per (sequence, head, run of chunks): warps 0-3 own the chunk's token rows (weights of the first sum, outputs),
+// warps 4-7 the state rows and the scaled x, warp 8 loads tiles with TMA, warp 9 issues the MMAs, warp 10 turns raw step
+// sizes into dt and L one chunk ahead.  When there are fewer heads than SMs the tokens are cut into segments: a first
+// launch computes what every segment adds to the state from zero, the second starts each segment from the combination.
+#include <algorithm>
+
+#include "sm100_common.cuh"
+#include "gb_layers.h"
+#include "tc_tiles.cuh"
+#include "layers_util.cuh"
+
+namespace gb {
+
+constexpr int SD_Q = 128;                  // tokens per chunk
+constexpr int SD_N = 128;                  // padded state size
+constexpr int SD_THREADS = 352;
+
+struct SsdParams {
+  int B, n, H, P, N, G, Ns;
+  const __nv_bfloat16* proj; long long ld_proj; int dt_col;
+  const float* dt_bias; const float* A_log; const float* D;
+  float* ssm;
+  __nv_bfloat16* y; long long ld_y;
+  const gb_seq_state* st;
+  int n_chunks, seg_chunks, n_seg, state_only;
+  float* ws_state;                         // [B, H, n_seg, P, Ns]: slot 0 = state before the call, slot k + 1 = segment k's part
+  float* ws_decay;                         // [B, H, n_seg]: log2 decay over segment k
+  int* status;
+};
+
+__device__ __forceinline__ float sd_ex2(float x) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+
+// 2 values -> packed bf16 pair and the packed remainders
+__device__ __forceinline__ void sd_split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = Cvt<__nv_bfloat16>::pack2(a, b);
+  const float2 h = Cvt<__nv_bfloat16>::unpack2(hi);
+  lo = Cvt<__nv_bfloat16>::pack2(a - h.x, b - h.y);
+}
+
+template <int PP>
+struct SsdCfg {
+  static constexpr int STAGES = PP == 64 ? 2 : 1;
+  static constexpr int NG = PP == 64 ? 2 : 1;                       // score buffers in tensor memory
+  static constexpr uint32_t TBC = SD_Q * SD_N * 2, TX = SD_Q * PP * 2, STAGE = 2 * TBC + TX;
+  static constexpr uint32_t TS = SD_N * PP * 2;
+  static constexpr size_t TILES = (size_t)STAGES * STAGE + 2 * TS + 2 * TX;
+  static constexpr size_t SMEM = TILES + 2 * 2 * SD_Q * 4 + 192;
+  static constexpr int COL_Y = 128 * NG, COL_Y2 = COL_Y + PP, COL_S = COL_Y2 + PP;
+};
+
+template <int PP>
+__global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_constant__ CUtensorMap tmX,
+                                                               const __grid_constant__ CUtensorMap tmB,
+                                                               const __grid_constant__ CUtensorMap tmC,
+                                                               const __grid_constant__ SsdParams p) {
+  using T = __nv_bfloat16;
+  using K = SsdCfg<PP>;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  if (smem_u32(smem) & 1023u) {            // no static shared memory: the dynamic window starts aligned
+    if (threadIdx.x == 0) atomicCAS(p.status, 0, ST_BAD_ARGUMENT);
+    return;
+  }
+  uint8_t* sShi = smem + K::STAGES * K::STAGE;
+  uint8_t* sSlo = sShi + K::TS;
+  uint8_t* sXhi = sSlo + K::TS;
+  uint8_t* sXlo = sXhi + K::TX;
+  float* sL = reinterpret_cast<float*>(sXlo + K::TX);       // [2][128] L in log2 units
+  float* sV = sL + 2 * SD_Q;                                // [2][128] log2(dt) - L
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * SD_Q);
+  uint64_t* full = bars;               // 2
+  uint64_t* empty = bars + 2;          // 2
+  uint64_t* l_full = bars + 4;         // 2
+  uint64_t* l_empty = bars + 6;        // 2
+  uint64_t* g_full = bars + 8;
+  uint64_t* m_ready = bars + 9;
+  uint64_t* y_full = bars + 10;
+  uint64_t* y_empty = bars + 11;
+  uint64_t* s_ready = bars + 12;
+  uint64_t* xw_ready = bars + 13;
+  uint64_t* s_full = bars + 14;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool so = p.state_only != 0;
+  const int seg = blockIdx.x % (so ? p.n_seg - 1 : p.n_seg), bh = blockIdx.x / (so ? p.n_seg - 1 : p.n_seg);
+  const int b = bh / p.H, h = bh - b * p.H, g = h / (p.H / p.G);
+  const int c_lo = seg * p.seg_chunks, c_hi = min(p.n_chunks, c_lo + p.seg_chunks), nc = c_hi - c_lo;
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], so ? 1 : 5);
+      mbar_init(&l_full[s], 1);
+      mbar_init(&l_empty[s], so ? 4 : 8);
+    }
+    mbar_init(g_full, 1);
+    mbar_init(m_ready, 4);
+    mbar_init(y_full, 1);
+    mbar_init(y_empty, 4);
+    mbar_init(s_ready, 4);
+    mbar_init(xw_ready, 4);
+    mbar_init(s_full, 1);
+    *abort_flag = 0;
+    fence_barrier_init();
+  }
+  if (warp == 9) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tm = *tmem_slot;
+  const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
+#define SD_WAIT(bar, ph, code) if (!at_wait(bar, ph, p.status, code, abort_flag)) break
+
+  if (warp == 8) {
+    // ------------------------------------------------------------------ TMA
+    if (lane == 0) {
+      for (int c = 0; c < nc; ++c) {
+        const int s = c % K::STAGES, ph = (c / K::STAGES) & 1;
+        SD_WAIT(&empty[s], ph ^ 1, ST_TIMEOUT_EMPTY);
+        uint8_t* st = smem + s * K::STAGE;
+        const int row = b * p.n + (c_lo + c) * SD_Q;
+        mbar_arrive_expect_tx(&full[s], so ? K::TBC + K::TX : K::STAGE);
+        load_tile<SD_N>(&tmB, &full[s], st + K::TBC, g * SD_N, row);
+        load_tile<PP>(&tmX, &full[s], st + 2 * K::TBC, h * PP, row);
+        if (!so) load_tile<SD_N>(&tmC, &full[s], st, g * SD_N, row);
+      }
+    }
+    __syncwarp();
+  } else if (warp == 9) {
+    // ------------------------------------------------------------------ MMA
+    if (lane == 0) {
+      const uint32_t id_g = make_idesc_f16(1, 0, 0, SD_Q, SD_Q);
+      const uint32_t id_y = make_idesc_f16(1, 0, 1, SD_Q, PP);
+      const uint32_t id_s = make_idesc_f16(1, 1, 1, SD_N, PP);
+      auto scores = [&](int c) {
+        const uint32_t st = smem_u32(smem + (c % K::STAGES) * K::STAGE);
+        mma_kmajor_kmajor<SD_N>(tm + (c % K::NG) * 128, st, st + K::TBC, id_g, false);
+        umma_commit(g_full);
+      };
+      bool ok = true;
+      if (!so) {
+        ok = at_wait(&full[0], 0, p.status, ST_TIMEOUT_FULL, abort_flag);
+        if (ok) { tc_fence_after(); scores(0); }
+      }
+      for (int c = 0; c < nc && ok; ++c) {
+        const int s = c % K::STAGES;
+        const uint32_t st = smem_u32(smem + s * K::STAGE), sx = st + 2 * K::TBC;
+        if (so) SD_WAIT(&full[s], (c / K::STAGES) & 1, ST_TIMEOUT_FULL);
+        SD_WAIT(s_ready, c & 1, ST_TIMEOUT_EMPTY);
+        if (!so) {
+          if (c > 0) SD_WAIT(y_empty, (c - 1) & 1, ST_TIMEOUT_TMEM_EMPTY);
+          tc_fence_after();
+          mma_kmajor_mnmajor<SD_N>(tm + K::COL_Y2, st, smem_u32(sShi), id_y, false);
+          mma_kmajor_mnmajor<SD_N>(tm + K::COL_Y2, st, smem_u32(sSlo), id_y, true);
+          SD_WAIT(m_ready, c & 1, ST_TIMEOUT_TMEM_EMPTY);
+          tc_fence_after();
+          const uint32_t m0 = tm + (c % K::NG) * 128;
+#pragma unroll
+          for (int part = 0; part < 2; ++part)
+#pragma unroll
+            for (int kk = 0; kk < SD_Q / 16; ++kk)
+              umma_f16_ts(tm + K::COL_Y, m0 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8,
+                          make_smem_desc_sw128(sx + kk * 2048, SD_Q * 128, 1024), id_y, (part || kk) ? 1u : 0u);
+          umma_commit(y_full);
+          if (K::STAGES == 2 && c + 1 < nc) {
+            SD_WAIT(&full[(c + 1) % K::STAGES], ((c + 1) / K::STAGES) & 1, ST_TIMEOUT_FULL);
+            tc_fence_after();
+            scores(c + 1);
+          }
+        }
+        SD_WAIT(xw_ready, c & 1, ST_TIMEOUT_EMPTY);
+        tc_fence_after();
+#pragma unroll
+        for (int part = 0; part < 2; ++part)
+#pragma unroll
+          for (int kk = 0; kk < SD_Q / 16; ++kk)
+            umma_f16(tm + K::COL_S, make_smem_desc_sw128(st + K::TBC + kk * 2048, SD_Q * 128, 1024),
+                     make_smem_desc_sw128(smem_u32(part ? sXlo : sXhi) + kk * 2048, SD_Q * 128, 1024), id_s, 1u);
+        umma_commit(s_full);
+        umma_commit(&empty[s]);
+        if (!so && K::STAGES == 1 && c + 1 < nc) {
+          SD_WAIT(y_full, c & 1, ST_TIMEOUT_TMEM_FULL);      // the one score buffer still holds this chunk's weights
+          SD_WAIT(&full[0], (c + 1) & 1, ST_TIMEOUT_FULL);
+          tc_fence_after();
+          scores(c + 1);
+        }
+      }
+    }
+    __syncwarp();
+  } else if (warp == 10) {
+    // ------------------------------------------------------------------ dt and L
+    const float bias = p.dt_bias[h], na2 = -expf(p.A_log[h]) * 1.4426950408889634f;
+    for (int c = 0; c < nc; ++c) {
+      const int s = c & 1, t0 = (c_lo + c) * SD_Q + lane * 4;
+      float dt[4], cum[4], run = 0.f;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        dt[k] = t0 + k < p.n ? ll_softplus(Cvt<T>::to_f(p.proj[((long long)b * p.n + t0 + k) * p.ld_proj + p.dt_col + h]) + bias) : 0.f;
+        run += na2 * dt[k];
+        cum[k] = run;
+      }
+      float inc = run;                                     // inclusive sum over lanes
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float v = __shfl_up_sync(0xffffffffu, inc, o);
+        if (lane >= o) inc += v;
+      }
+      const float before = inc - run;
+      SD_WAIT(&l_empty[s], ((c >> 1) & 1) ^ 1, ST_TIMEOUT_EMPTY);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float L = before + cum[k];
+        sL[s * SD_Q + lane * 4 + k] = L;
+        sV[s * SD_Q + lane * 4 + k] = log2f(dt[k]) - L;
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&l_full[s]);
+    }
+    __syncwarp();
+  } else if (warp < 4) {
+    // ------------------------------------------------------------------ token rows
+    const int r = threadIdx.x;
+    const float D = p.D[h];
+    for (int c = 0; c < nc && !so; ++c) {
+      const int ls = c & 1, s = c % K::STAGES, t = (c_lo + c) * SD_Q + r;
+      SD_WAIT(&l_full[ls], (c >> 1) & 1, ST_TIMEOUT_FULL);
+      const float L = sL[ls * SD_Q + r];
+      const float4* v4 = reinterpret_cast<const float4*>(sV + ls * SD_Q);
+      const uint32_t tg = tm + (c % K::NG) * 128 + lane_base;
+      SD_WAIT(g_full, c & 1, ST_TIMEOUT_TMEM_FULL);
+      tc_fence_after();
+      // weights (C_t . B_s) exp(L_t - L_s) dt_s, written over the scores they come from: per 32 columns, 16 columns of
+      // packed values and 16 of packed remainders
+#pragma unroll 1
+      for (int q = 0; q < 4; ++q) {
+        uint32_t hi[16], lo[16];
+        if (q <= warp) {
+          uint32_t rg[32];
+          tmem_ld_32x32(tg + q * 32, rg);
+          tmem_ld_wait();
+#pragma unroll
+          for (int k = 0; k < 8; ++k) {
+            const float4 v = v4[q * 8 + k];
+            float m[4];
+            m[0] = __uint_as_float(rg[4 * k]) * sd_ex2(fminf(L + v.x, 126.f));
+            m[1] = __uint_as_float(rg[4 * k + 1]) * sd_ex2(fminf(L + v.y, 126.f));
+            m[2] = __uint_as_float(rg[4 * k + 2]) * sd_ex2(fminf(L + v.z, 126.f));
+            m[3] = __uint_as_float(rg[4 * k + 3]) * sd_ex2(fminf(L + v.w, 126.f));
+            if (q == warp) {
+#pragma unroll
+              for (int e = 0; e < 4; ++e)
+                if (4 * k + e > lane) m[e] = 0.f;
+            }
+            sd_split2(m[0], m[1], hi[2 * k], lo[2 * k]);
+            sd_split2(m[2], m[3], hi[2 * k + 1], lo[2 * k + 1]);
+          }
+        } else {
+#pragma unroll
+          for (int k = 0; k < 16; ++k) { hi[k] = 0u; lo[k] = 0u; }
+        }
+        tmem_st_32x16(tg + q * 32, hi);
+        tmem_st_32x16(tg + q * 32 + 16, lo);
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(m_ready);
+      const float eL = sd_ex2(L);
+      SD_WAIT(y_full, c & 1, ST_TIMEOUT_TMEM_FULL);
+      SD_WAIT(&full[s], (c / K::STAGES) & 1, ST_TIMEOUT_FULL);      // long since true; this thread reads x itself
+      tc_fence_after();
+      const uint8_t* sx = smem + s * K::STAGE + 2 * K::TBC;
+      T* yp = p.y + ((long long)b * p.n + t) * p.ld_y + h * p.P;
+      const bool live = t < p.n;
+      const bool vec = p.P == PP && ((reinterpret_cast<uintptr_t>(p.y) | (uintptr_t)(p.ld_y * 2)) & 15) == 0;
+#pragma unroll
+      for (int q = 0; q < PP / 32; ++q) {
+        uint32_t a[32], e[32];
+        tmem_ld_32x32(tm + K::COL_Y + lane_base + q * 32, a);
+        tmem_ld_32x32(tm + K::COL_Y2 + lane_base + q * 32, e);
+        tmem_ld_wait();
+#pragma unroll
+        for (int k = 0; k < 4 && live; ++k) {
+          const int col = q * 32 + 8 * k;
+          const uint4 xq = *reinterpret_cast<const uint4*>(sx + (col >> 6) * (SD_Q * 128) + sw128_off(r, col & 63));
+          const uint32_t xw[4] = {xq.x, xq.y, xq.z, xq.w};
+          float v[8];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float2 x = Cvt<T>::unpack2(xw[j]);
+            v[2 * j] = __uint_as_float(a[8 * k + 2 * j]) + eL * __uint_as_float(e[8 * k + 2 * j]) + D * x.x;
+            v[2 * j + 1] = __uint_as_float(a[8 * k + 2 * j + 1]) + eL * __uint_as_float(e[8 * k + 2 * j + 1]) + D * x.y;
+          }
+          if (vec) {
+            uint4 o;
+            o.x = Cvt<T>::pack2(v[0], v[1]); o.y = Cvt<T>::pack2(v[2], v[3]);
+            o.z = Cvt<T>::pack2(v[4], v[5]); o.w = Cvt<T>::pack2(v[6], v[7]);
+            *reinterpret_cast<uint4*>(yp + col) = o;
+          } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+              if (col + j < p.P) yp[col + j] = Cvt<T>::from_f(v[j]);
+          }
+        }
+        __syncwarp();                       // the next tensor-memory load is the whole warp's
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) { mbar_arrive(y_empty); mbar_arrive(&empty[s]); mbar_arrive(&l_empty[ls]); }
+    }
+  } else {
+    // ------------------------------------------------------------------ state rows and scaled x
+    const int r = threadIdx.x - 128;            // state column (0 .. 127) / token of the chunk
+    const bool live_n = r < p.N;
+    const long long per = (long long)p.P * p.Ns;
+    float* home = p.ssm + bh * per;
+    float* ws = p.ws_state ? p.ws_state + (long long)bh * p.n_seg * per : nullptr;
+    const uint32_t ts = tm + K::COL_S + lane_base;
+    const bool fresh = p.st[b].abs_pos == 0;
+    // the state this run starts from
+#pragma unroll 1
+    for (int q = 0; q < PP / 16; ++q) {
+      uint32_t v[16];
+#pragma unroll
+      for (int k = 0; k < 16; ++k) {
+        const int pp = q * 16 + k;
+        float x = 0.f;
+        if (live_n && pp < p.P) {
+          const long long at = (long long)pp * p.Ns + r;
+          if (so) {
+            if (seg == 0) ws[at] = fresh ? 0.f : home[at];          // the second launch's last segment replaces `home`
+          } else if (p.n_seg == 1) {
+            x = fresh ? 0.f : home[at];
+          } else {
+            x = ws[at];
+            for (int j = 0; j < seg; ++j) x = x * sd_ex2(p.ws_decay[(long long)bh * p.n_seg + j]) + ws[(j + 1) * per + at];
+          }
+        }
+        v[k] = __float_as_uint(x);
+      }
+      __syncwarp();
+      tmem_st_32x16(ts + q * 16, v);
+    }
+    tmem_st_wait();
+    float total = 0.f;
+    bool ok = true;
+    for (int c = 0; c < nc; ++c) {
+      const int ls = c & 1, s = c % K::STAGES;
+      ok = false;
+      SD_WAIT(&l_full[ls], (c >> 1) & 1, ST_TIMEOUT_FULL);
+      const float Ll = sL[ls * SD_Q + SD_Q - 1], dec = sd_ex2(Ll), w = sd_ex2(fminf(Ll + sV[ls * SD_Q + r], 126.f));
+      total += Ll;
+      if (c > 0) SD_WAIT(s_full, (c - 1) & 1, ST_TIMEOUT_TMEM_FULL);
+      tc_fence_after();
+#pragma unroll
+      for (int q = 0; q < PP / 16; ++q) {
+        uint32_t v[16];
+        tmem_ld_32x16(ts + q * 16, v);
+        tmem_ld_wait();
+        if (!so) {
+#pragma unroll
+          for (int k = 0; k < 2; ++k) {
+            uint4 hi, lo;
+            sd_split2(__uint_as_float(v[8 * k]), __uint_as_float(v[8 * k + 1]), hi.x, lo.x);
+            sd_split2(__uint_as_float(v[8 * k + 2]), __uint_as_float(v[8 * k + 3]), hi.y, lo.y);
+            sd_split2(__uint_as_float(v[8 * k + 4]), __uint_as_float(v[8 * k + 5]), hi.z, lo.z);
+            sd_split2(__uint_as_float(v[8 * k + 6]), __uint_as_float(v[8 * k + 7]), hi.w, lo.w);
+            const int col = q * 16 + 8 * k;
+            const uint32_t off = (col >> 6) * (SD_N * 128) + sw128_off(r, col & 63);
+            *reinterpret_cast<uint4*>(sShi + off) = hi;
+            *reinterpret_cast<uint4*>(sSlo + off) = lo;
+          }
+        }
+#pragma unroll
+        for (int k = 0; k < 16; ++k) v[k] = __float_as_uint(__uint_as_float(v[k]) * dec);
+        tmem_st_32x16(ts + q * 16, v);
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      fence_proxy_async();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(s_ready);
+      SD_WAIT(&full[s], (c / K::STAGES) & 1, ST_TIMEOUT_FULL);
+      const uint8_t* sx = smem + s * K::STAGE + 2 * K::TBC;
+#pragma unroll
+      for (int q = 0; q < PP / 8; ++q) {
+        const uint32_t off = (q >> 3) * (SD_Q * 128) + sw128_off(r, (q & 7) * 8);
+        const uint4 xq = *reinterpret_cast<const uint4*>(sx + off);
+        const uint32_t xw[4] = {xq.x, xq.y, xq.z, xq.w};
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 x = Cvt<T>::unpack2(xw[j]);
+          sd_split2(x.x * w, x.y * w, hi[j], lo[j]);
+        }
+        *reinterpret_cast<uint4*>(sXhi + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(sXlo + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      }
+      fence_proxy_async();
+      __syncwarp();
+      if (lane == 0) { mbar_arrive(xw_ready); mbar_arrive(&l_empty[ls]); }
+      ok = true;
+    }
+    if (ok && nc > 0 && at_wait(s_full, (nc - 1) & 1, p.status, ST_TIMEOUT_TMEM_FULL, abort_flag)) {
+      tc_fence_after();
+      float* dst = so ? ws + (seg + 1) * per : (seg == p.n_seg - 1 ? home : nullptr);
+#pragma unroll 1
+      for (int q = 0; q < PP / 16; ++q) {
+        uint32_t v[16];
+        tmem_ld_32x16(ts + q * 16, v);
+        tmem_ld_wait();
+        if (dst && live_n) {
+#pragma unroll
+          for (int k = 0; k < 16; ++k)
+            if (q * 16 + k < p.P) dst[(long long)(q * 16 + k) * p.Ns + r] = __uint_as_float(v[k]);
+        }
+        __syncwarp();
+      }
+      if (so && r == 0) p.ws_decay[(long long)bh * p.n_seg + seg] = total;
+      tc_fence_before();
+    }
+  }
+#undef SD_WAIT
+  __syncthreads();
+  if (*abort_flag) {
+    for (int k = 0; k < 64; ++k) __nanosleep(1000);
+    __syncthreads();
+  }
+  if (warp == 9) { tc_fence_after(); tmem_dealloc(tm, 512); }
+}
+
+struct SsdPlan { int n_chunks, seg_chunks, n_seg; };
+
+// Segments per head: the cheapest number of rounds over the SMs, where cutting at all costs the extra state pass.
+static SsdPlan ssd_plan(int BH, int n, int sms) {
+  SsdPlan best{(n + SD_Q - 1) / SD_Q, 0, 1};
+  best.seg_chunks = best.n_chunks;
+  double cost = (double)((BH + sms - 1) / sms) * best.n_chunks;
+  for (int s = 2; s <= 16 && s <= best.n_chunks; ++s) {
+    const int per = (best.n_chunks + s - 1) / s, k = (best.n_chunks + per - 1) / per;
+    const double c = per * ((double)((BH * k + sms - 1) / sms) + 0.5 * ((BH * (k - 1) + sms - 1) / sms)) + 3.0;
+    if (c < cost * 0.95) { cost = c; best.seg_chunks = per; best.n_seg = k; }
+  }
+  return best;
+}
+
+static int ssd_sms() {
+  static int sms = 0;
+  if (!sms) {
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) sms = 0;
+  }
+  return sms;
+}
+
+template <int PP>
+static int ssd_go(const gb_ll_mamba_args& a, int force_segments, cudaStream_t st) {
+  using K = SsdCfg<PP>;
+  static_assert(K::SMEM <= 232448 && K::COL_S + PP <= 512, "shared memory / tensor memory budget");
+  const int sms = ssd_sms();
+  if (sms <= 0) return -10;
+  static bool attr = false;
+  if (!attr) {
+    if (cudaFuncSetAttribute(ll_ssd_kernel<PP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)K::SMEM) != cudaSuccess) return -10;
+    attr = true;
+  }
+  CUtensorMap tx, tb, tc;
+  const uint64_t rows = (uint64_t)a.B * a.n;
+  if (gb_make_tmap_2d_16b(&tx, a.xh, rows, (uint64_t)a.H * PP, (uint64_t)a.H * PP, SD_Q, 64, 1)) return -20;
+  if (gb_make_tmap_2d_16b(&tb, a.bc, rows, (uint64_t)a.G * SD_N, (uint64_t)a.G * SD_N, SD_Q, 64, 1)) return -21;
+  if (gb_make_tmap_2d_16b(&tc, a.cc, rows, (uint64_t)a.G * SD_N, (uint64_t)a.G * SD_N, SD_Q, 64, 1)) return -22;
+  SsdPlan plan = ssd_plan(a.B * a.H, a.n, sms);
+  if (force_segments > 0) {
+    const int per = (plan.n_chunks + force_segments - 1) / force_segments;
+    plan.seg_chunks = per;
+    plan.n_seg = (plan.n_chunks + per - 1) / per;
+  }
+  if (!a.chunk_ws) { plan.n_seg = 1; plan.seg_chunks = plan.n_chunks; }
+  SsdParams p{};
+  p.B = a.B; p.n = a.n; p.H = a.H; p.P = a.P; p.N = a.N; p.G = a.G; p.Ns = a.Ns;
+  p.proj = static_cast<const __nv_bfloat16*>(a.proj); p.ld_proj = a.ld_proj; p.dt_col = 2 * a.H * a.P + 2 * a.G * a.N;
+  p.dt_bias = a.dt_bias; p.A_log = a.A_log; p.D = a.D; p.ssm = a.ssm;
+  p.y = static_cast<__nv_bfloat16*>(a.y); p.ld_y = a.ld_y; p.st = a.st; p.status = a.status;
+  p.n_chunks = plan.n_chunks; p.seg_chunks = plan.seg_chunks; p.n_seg = plan.n_seg;
+  const long long BH = (long long)a.B * a.H;
+  if (plan.n_seg > 1) {
+    p.ws_state = a.chunk_ws;
+    p.ws_decay = a.chunk_ws + BH * plan.n_seg * a.P * a.Ns;
+    p.state_only = 1;
+    ll_ssd_kernel<PP><<<(unsigned)(BH * (plan.n_seg - 1)), SD_THREADS, K::SMEM, st>>>(tx, tb, tc, p);
+    p.state_only = 0;
+  }
+  ll_ssd_kernel<PP><<<(unsigned)(BH * plan.n_seg), SD_THREADS, K::SMEM, st>>>(tx, tb, tc, p);
+  return gb_launch_rc();
+}
+
+}  // namespace gb
+
+using namespace gb;
+
+extern "C" int gb_ll_ssd_ok(const gb_ll_mamba_args* p) {
+  if (!p || p->dtype != 1) return -1;
+  if ((p->Pp != 64 && p->Pp != 128) || p->Np != SD_N || p->P > p->Pp || p->N > p->Np) return -2;
+  if ((long long)p->B * p->n > 0x7fffffffll) return -3;
+  return 0;
+}
+
+extern "C" long long gb_ll_ssd_ws_floats(int B, int H, int P, int Ns, int n, int segments) {
+  int k = segments;
+  if (k <= 0) {
+    const int sms = ssd_sms();
+    k = ssd_plan(B * H, n, sms > 0 ? sms : 148).n_seg;
+  }
+  return k > 1 ? (long long)B * H * k * ((long long)P * Ns + 1) : 0;
+}
+
+extern "C" int gb_ll_ssd(const gb_ll_mamba_args* p, int segments, cudaStream_t st) {
+  if (const int rc = gb_ll_ssd_ok(p)) return rc;
+  if (!p->st || !p->proj || !p->xh || !p->bc || !p->cc || !p->y || !p->ssm || !p->status || !p->dt_bias || !p->A_log || !p->D ||
+      p->B <= 0 || p->n <= 0 || p->G <= 0 || p->H % p->G || p->Ns < p->N) return -1;
+  return p->Pp == 64 ? ssd_go<64>(*p, segments, st) : ssd_go<128>(*p, segments, st);
+}

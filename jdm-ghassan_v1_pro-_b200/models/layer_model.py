@@ -26,6 +26,9 @@ from ..utils import canary as CA
 from .layer_list import AttentionMixer, LayerListConfig, Mamba2Mixer, check_tensors
 
 
+SSD_MIN_TOKENS = 17       # shorter portions take the token-by-token recurrence: a chunk is 128 tokens however few are real
+
+
 def _up(n: int, a: int) -> int:
     return (n + a - 1) // a * a
 
@@ -118,6 +121,13 @@ class LayerModel:
             self._bufs[key] = t
         return t
 
+    def _scratch(self, name: str, floats: int) -> torch.Tensor:
+        t = self._bufs.get((name,))
+        if t is None or t.numel() < floats:
+            t = torch.empty(floats, dtype=torch.float32, device=self.dev)
+            self._bufs[(name,)] = t
+        return t
+
     # ------------------------------------------------------------------ products over rows
     def _gemm(self, a, w, out, rows):
         """out[:rows] = a[:rows] @ w^T; ``out`` in the compute type or fp32."""
@@ -175,8 +185,8 @@ class LayerModel:
         a = K.MambaArgs()
         a.dtype, a.B, a.n = K.DTYPE[self.dtype], B, n
         a.H, a.P, a.N, a.G, a.taps = m.heads, m.vdim, m.state, m.groups, m.conv
-        pad = 64 if self.dtype == torch.bfloat16 else 8
-        a.Pp, a.Np, a.Ns = _up(m.vdim, pad), _up(m.state, pad), state.ns
+        padx, padn = (64, 128) if self.dtype == torch.bfloat16 else (8, 8)      # whole tiles for the chunked recurrence
+        a.Pp, a.Np, a.Ns = _up(m.vdim, padx), _up(m.state, padn), state.ns
         proj = self.buf("proj", _up(w.w_in.shape[0], 8))
         a.proj, a.ld_proj = proj.data_ptr(), proj.stride(0)
         v = w.vec
@@ -214,7 +224,14 @@ class LayerModel:
                 K.mamba_step(a)
             else:
                 K.conv(a)
-                K.scan(a)
+                if self.use_tc and n >= SSD_MIN_TOKENS and K.ssd_ok(a):
+                    need = K.ssd_ws_floats(B, a.H, a.P, a.Ns, n)
+                    if need:
+                        a.chunk_ws = self._scratch("ssd", need).data_ptr()
+                        self.launches += 1
+                    K.ssd(a)
+                else:
+                    K.scan(a)
                 self.launches += 1
             K.gated_norm(a)
             self.launches += 2

@@ -106,7 +106,7 @@ def attn_prefill(a: AttnArgs):
 
 
 def attn_tc_ok(a: AttnArgs) -> bool:
-    return hasattr(_lib.lib(), 'gb_ll_attn_tc_ok') and _lib.lib().gb_ll_attn_tc_ok(ctypes.byref(a)) == 0
+    return _lib.lib().gb_ll_attn_tc_ok(ctypes.byref(a)) == 0
 
 
 def attn_tc(a: AttnArgs):
@@ -123,6 +123,21 @@ def conv(a: MambaArgs):
 
 def scan(a: MambaArgs):
     _call("gb_ll_scan", ctypes.byref(a))
+
+
+def ssd_ok(a: MambaArgs) -> bool:
+    return _lib.lib().gb_ll_ssd_ok(ctypes.byref(a)) == 0
+
+
+def ssd_ws_floats(B, H, P, Ns, n, segments=0) -> int:
+    f = _lib.lib().gb_ll_ssd_ws_floats
+    f.restype = c_ll
+    return int(f(c_int(B), c_int(H), c_int(P), c_int(Ns), c_int(n), c_int(segments)))
+
+
+def ssd(a: MambaArgs, segments=0):
+    """The recurrence in chunks on the tensor cores; ``segments``: runs a sequence is cut into (0: by the machine)."""
+    _lib.check_rc(_lib.lib().gb_ll_ssd(ctypes.byref(a), c_int(segments), _lib.stream_ptr()), "gb_ll_ssd")
 
 
 def mamba_step(a: MambaArgs):

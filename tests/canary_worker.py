@@ -85,6 +85,23 @@ training:
         eng.decode_steps(30, sp)                               # past the cache size: the ring wraps
         torch.cuda.synchronize()
         bad += ["decode/%s/%s" % (kw, b) for b in CA.check()]
+    # layer-list models: prompt passes, portions, both token steps, in both precisions
+    import layers_cases as LC
+    from ghassan_b200.inference.layer_engine import LayerEngine
+    from ghassan_b200.models.layer_list import LayerListConfig
+    for name, raw in sorted(LC.cases().items()):
+        for dtype in (torch.bfloat16, torch.float32):
+            for B in (1, 9):
+                eng = LayerEngine(LayerListConfig.from_json(raw), LC.weights(raw), batch=B, max_len=400, prefill_chunk=70, dtype=dtype)
+                eng.reset(1)
+                eng.prefill(torch.tensor([LC.tokens(raw, 151, b) for b in range(B)], dtype=torch.int32))
+                sp = SamplingParams(seed=3, top_k=20)
+                eng.sample_first(sp)
+                eng.decode_steps(20, sp)
+                eng.reset(1)
+                eng.step("a", LC.tokens(raw, 33), [0, 32])
+                torch.cuda.synchronize()
+                bad += ["layers/%s/%s/%d/%s" % (name, dtype, B, b) for b in CA.check()]
     if bad:
         print("CANARIES HIT", bad, flush=True)
         return 1

@@ -51,9 +51,6 @@ __device__ __forceinline__ void load8(const uint8_t* __restrict__ row, int u, fl
       w[i] = d * (float)(int8_t)((vx >> (8 * i)) & 0xFF);
       w[4 + i] = d * (float)(int8_t)((vy >> (8 * i)) & 0xFF);
     }
-  } else if constexpr (FMT == GB_W_F32) {
-    const float4 a = reinterpret_cast<const float4*>(row)[2 * (size_t)u], b = reinterpret_cast<const float4*>(row)[2 * (size_t)u + 1];
-    w[0] = a.x; w[1] = a.y; w[2] = a.z; w[3] = a.w; w[4] = b.x; w[5] = b.y; w[6] = b.z; w[7] = b.w;
   } else {   // GB_W_Q4_1
     const uint8_t* p = row + (size_t)(u >> 2) * 20;
     const float d = h2f(ld_u16(p)), m = h2f(ld_u16(p + 2));

@@ -41,6 +41,7 @@ int gb_ll_advance(gb_seq_state* state, int* pos_out, int B, int n, cudaStream_t 
 //   prologue 1: x_new = x + norm(y) * w1 (y NULL: x_new = x), written to x_out by one block; v = x_new, or
 //               norm(x_new) * w2 when w2 is given
 //   prologue 2: v = norm_parts(y16 * silu(z16)) * w1, `parts` equal parts each by its own root mean square
+//   prologue 3: the same from v32 = y silu(z) (fp32, pitch d) and `n_sq` sums of squares per sequence, n_sq / parts to a part
 // swiglu != 0: W holds gate/up rows interleaved in blocks of 64 (N = 2 E rows) and out[b, j] = silu(gate_j) * up_j.
 // softcap > 0: out = cap * tanh(out / cap).
 typedef struct gb_ll_gemv_args {
@@ -50,6 +51,7 @@ typedef struct gb_ll_gemv_args {
   const void* x16; long long ldx;
   const float* x; const float* y; long long ldy; const float* w1; const float* w2; float eps; float* x_out;
   const void* y16; long long ldy16; const void* z16; long long ldz; int parts;
+  const float* v32; const float* sq; int n_sq;
   void* out; long long ldo; int out_f32; float softcap;
 } gb_ll_gemv_args;
 int gb_ll_gemv(const gb_ll_gemv_args* a, cudaStream_t st);
@@ -64,6 +66,8 @@ typedef struct gb_ll_attn_args {
   int dk, dv, dkp, dvp;                  // head sizes and their padded row lengths in q and the caches (padding is zero)
   int rot_dims, rot_half;                // rotated leading dimensions; 0: pairs (2i, 2i+1), 1: pairs (i, i + rot_dims/2)
   const double* freq;                    // [rot_dims / 2] angular frequencies
+  const float* cs;                       // optional [rows, rot_dims / 2, 2]: cosines and sines of this call's rows
+                                         // (gb_ll_rotations); NULL: computed on the spot
   int qk_norm;                           // divide q and k by their root mean square after the rotation
   float eps, scale;
   int window, keep, cap;
@@ -78,6 +82,7 @@ typedef struct gb_ll_attn_args {
   int pos0_max;                          // host's upper bound of abs_pos over the B sequences (tile counts); -1 unknown
   int* status;
 } gb_ll_attn_args;
+int gb_ll_rotations(const double* freq, int pairs, const gb_seq_state* st, int B, int n, float* cs, cudaStream_t stream);
 int gb_ll_qkv_store(const gb_ll_attn_args* a, cudaStream_t st);     // rotation, norm, q out, k and v into the cache
 int gb_ll_attn_prefill(const gb_ll_attn_args* a, cudaStream_t st);  // any dtype and head size up to 256
 int gb_ll_attn_tc_ok(const gb_ll_attn_args* a);                     // 0 when the tensor-core kernel covers the shapes
@@ -99,6 +104,8 @@ typedef struct gb_ll_mamba_args {
   void* xh; void* bc; void* cc;          // convolved: [rows, H, Pp], [rows, G, Np], [rows, G, Np]
   void* y; long long ld_y;               // [rows, H*P]
   void* out; long long ld_out;           // [rows, H*P] gated and normed
+  float* gated; float* gated_sq;         // token step, optional: y silu(z) [B, H*P] and its sums of squares [B, H, ceil(P/32)]
+                                         // instead of y
   const gb_seq_state* st;
   float* chunk_ws;                       // chunked scan: gb_ll_ssd_ws_floats floats, or NULL (no cutting into segments)
   int* status;

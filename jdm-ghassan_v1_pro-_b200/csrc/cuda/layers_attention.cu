@@ -9,6 +9,72 @@
 
 namespace gb {
 
+// Angle of a pair at a position: the product in double, reduced to one turn, then an fp32 cosine and sine.
+__device__ __forceinline__ float2 ll_rotation(int pos, double freq) {
+  double ang = (double)pos * freq;
+  ang -= 6.283185307179586476925 * rint(ang * 0.159154943091895335769);
+  float sn, cs;
+  sincosf((float)ang, &sn, &cs);
+  return make_float2(cs, sn);
+}
+
+__global__ void __launch_bounds__(256) ll_rotations_kernel(const double* __restrict__ freq, int pairs, const gb_seq_state* __restrict__ st,
+                                                           int n, long long total, float2* __restrict__ cs) {
+  pdl_wait();
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i >= total) return;
+  const int r = (int)(i / pairs), b = r / n;
+  cs[i] = ll_rotation(st[b].abs_pos + r - b * n, freq[i - (long long)r * pairs]);
+}
+
+// LPH lanes per head, eight dimensions per lane (head sizes and offsets in multiples of eight, interleaved pairs).
+template <typename T, int LPH>
+__global__ void __launch_bounds__(256) ll_qkv_store_vec_kernel(const __grid_constant__ gb_ll_attn_args a) {
+  pdl_wait();
+  const int heads = a.H + 2 * a.G;
+  const int lane = threadIdx.x & 31, sub = lane % LPH, c = sub * 8;
+  const long long item = (blockIdx.x * 8LL + (threadIdx.x >> 5)) * (32 / LPH) + lane / LPH;
+  const bool live = item < (long long)a.B * a.n * heads;
+  const int r = live ? (int)(item / heads) : 0, h = live ? (int)(item - (long long)r * heads) : 0;
+  const int b = r / a.n, pos = a.st[b].abs_pos + r - b * a.n;
+  const T* row = reinterpret_cast<const T*>(a.proj) + r * a.ld_proj;
+  const long long crow = (long long)b * a.cap + ll_ring_row(pos, a.keep, a.cap);
+  const bool is_v = h >= a.H + a.G;
+  const int d = is_v ? a.dv : a.dk, dp = is_v ? a.dvp : a.dkp;
+  const T* src = is_v ? row + (a.H + a.G) * a.dk + (h - a.H - a.G) * a.dv : row + h * a.dk;
+  T* dst = is_v ? reinterpret_cast<T*>(a.cache_v) + (crow * a.G + (h - a.H - a.G)) * a.dvp
+                : h < a.H ? reinterpret_cast<T*>(a.q) + ((long long)r * a.H + h) * a.dkp
+                          : reinterpret_cast<T*>(a.cache_k) + (crow * a.G + (h - a.H)) * a.dkp;
+  float v[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] = 0.f;
+  if (live && c < d) ll_load8(src + c, v);
+  float ss = 0.f;
+  if (!is_v) {
+    if (c < a.rot_dims) {
+      const float4* cs = reinterpret_cast<const float4*>(a.cs + (long long)r * a.rot_dims + c);
+      const float4 p0 = cs[0], p1 = cs[1];
+      const float cc[4] = {p0.x, p0.z, p1.x, p1.z}, sn[4] = {p0.y, p0.w, p1.y, p1.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float x = v[2 * e], y = v[2 * e + 1];
+        v[2 * e] = x * cc[e] - y * sn[e];
+        v[2 * e + 1] = y * cc[e] + x * sn[e];
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += v[e] * v[e];
+  }
+#pragma unroll
+  for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (!is_v && a.qk_norm) {
+    const float inv = ll_inv_rms(ss, a.dk, a.eps);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= inv;
+  }
+  if (live && c < dp) ll_store8(dst + c, v);
+}
+
 // One warp per (row, head) over the query, key and value heads of the fused projection.
 template <typename T>
 __global__ void __launch_bounds__(256) ll_qkv_store_kernel(const __grid_constant__ gb_ll_attn_args a) {
@@ -47,12 +113,8 @@ __global__ void __launch_bounds__(256) ll_qkv_store_kernel(const __grid_constant
         const bool second = a.rot_half ? i >= half : (i & 1);
         const int pi = a.rot_half ? (second ? i - half : i + half) : i ^ 1;
         const float xp = Cvt<T>::to_f(src[pi]);
-        // angle in double, reduced to one turn, then an fp32 sine and cosine
-        double ang = (double)pos * a.freq[pair];
-        ang -= 6.283185307179586476925 * rint(ang * 0.159154943091895335769);
-        float sn, cs;
-        sincosf((float)ang, &sn, &cs);
-        x = second ? x * cs + xp * sn : x * cs - xp * sn;
+        const float2 cs = a.cs ? reinterpret_cast<const float2*>(a.cs)[(long long)r * half + pair] : ll_rotation(pos, a.freq[pair]);
+        x = second ? x * cs.x + xp * cs.y : x * cs.x - xp * cs.y;
       }
       v[k] = x;
       ss += x * x;
@@ -201,25 +263,48 @@ __global__ void __launch_bounds__(128) ll_attn_decode_kernel(const __grid_consta
     for (int e = 0; e < EPL; ++e) { q[x][e] = 0.f; o[x][e] = 0.f; }
     if (x < nh && kl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.q) + ((long long)b * a.H + h0 + x) * a.dkp + lane * EPL, q[x]);
   }
-  for (int e0 = lo + warp; e0 < hi; e0 += 4) {
-    const int p = e0 < kr.n_kept ? e0 : kr.win_lo + (e0 - kr.n_kept);
-    const long long crow = ((long long)b * a.cap + ll_ring_row(p, a.keep, a.cap)) * a.G + g;
-    float kf[EPL], vf[EPL];
+  constexpr int KB = EPL <= 4 ? 4 : 2;            // keys in flight per warp: all their loads come before the first use
+  for (int e0 = lo + warp * KB; e0 < hi; e0 += 4 * KB) {
+    float kf[KB][EPL], vf[KB][EPL];
 #pragma unroll
-    for (int e = 0; e < EPL; ++e) { kf[e] = 0.f; vf[e] = 0.f; }
-    if (kl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.cache_k) + crow * a.dkp + lane * EPL, kf);
-    if (vl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.cache_v) + crow * a.dvp + lane * EPL, vf);
+    for (int j = 0; j < KB; ++j) {
+      const int e = min(e0 + j, hi - 1);
+      const int p = e < kr.n_kept ? e : kr.win_lo + (e - kr.n_kept);
+      const long long crow = ((long long)b * a.cap + ll_ring_row(p, a.keep, a.cap)) * a.G + g;
+#pragma unroll
+      for (int x = 0; x < EPL; ++x) { kf[j][x] = 0.f; vf[j][x] = 0.f; }
+      if (kl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.cache_k) + crow * a.dkp + lane * EPL, kf[j]);
+      if (vl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.cache_v) + crow * a.dvp + lane * EPL, vf[j]);
+    }
 #pragma unroll
     for (int x = 0; x < GQ; ++x) {
-      float s = 0.f;
+      float s[KB], mn = m[x];
 #pragma unroll
-      for (int e = 0; e < EPL; ++e) s += q[x][e] * kf[e];
-      s = warp_sum(s) * a.scale;
-      const float mn = fmaxf(m[x], s);
-      const float c = expf(m[x] - mn), pr = expf(s - mn);
-      l[x] = l[x] * c + pr;
+      for (int j = 0; j < KB; ++j) {
+        s[j] = 0.f;
 #pragma unroll
-      for (int e = 0; e < EPL; ++e) o[x][e] = o[x][e] * c + pr * vf[e];
+        for (int e = 0; e < EPL; ++e) s[j] += q[x][e] * kf[j][e];
+      }
+#pragma unroll
+      for (int d = 16; d > 0; d >>= 1)
+#pragma unroll
+        for (int j = 0; j < KB; ++j) s[j] += __shfl_xor_sync(0xffffffffu, s[j], d);
+#pragma unroll
+      for (int j = 0; j < KB; ++j) {
+        s[j] = e0 + j < hi ? s[j] * a.scale : -INFINITY;
+        mn = fmaxf(mn, s[j]);
+      }
+      const float c = expf(m[x] - mn);            // the first key of a group is always real, so mn is finite
+      l[x] *= c;
+#pragma unroll
+      for (int e = 0; e < EPL; ++e) o[x][e] *= c;
+#pragma unroll
+      for (int j = 0; j < KB; ++j) {
+        const float pr = expf(s[j] - mn);
+        l[x] += pr;
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) o[x][e] += pr * vf[j][e];
+      }
       m[x] = mn;
     }
   }
@@ -327,9 +412,28 @@ static int ll_attn_check(const gb_ll_attn_args* p) {
   return p->dtype == 1 || p->dtype == 2 ? 0 : -6;
 }
 
+extern "C" int gb_ll_rotations(const double* freq, int pairs, const gb_seq_state* st, int B, int n, float* cs, cudaStream_t stream) {
+  if (!freq || !st || !cs || pairs <= 0 || B <= 0 || n <= 0) return -1;
+  const long long total = (long long)B * n * pairs;
+  GB_PDL_LAUNCH(ll_rotations_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), stream, freq, pairs, st, n, total, reinterpret_cast<float2*>(cs));
+  return gb_launch_rc();
+}
+
 extern "C" int gb_ll_qkv_store(const gb_ll_attn_args* p, cudaStream_t st) {
   if (const int rc = ll_attn_check(p)) return rc;
   const long long items = (long long)p->B * p->n * (p->H + 2 * p->G);
+  const bool vec = p->dk % 8 == 0 && p->dv % 8 == 0 && p->rot_dims % 8 == 0 && !p->rot_half && (p->cs || p->rot_dims == 0) && p->ld_proj % 8 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(p->proj) | reinterpret_cast<uintptr_t>(p->q) | reinterpret_cast<uintptr_t>(p->cache_k) |
+                     reinterpret_cast<uintptr_t>(p->cache_v) | reinterpret_cast<uintptr_t>(p->cs)) & 15) == 0;
+  if (vec) {
+    const int hd = p->dkp > p->dvp ? p->dkp : p->dvp, lph = hd <= 64 ? 8 : hd <= 128 ? 16 : 32;
+    const dim3 vg((unsigned)((items + 8 * (32 / lph) - 1) / (8 * (32 / lph))));
+#define QV(T, L) GB_PDL_LAUNCH((ll_qkv_store_vec_kernel<T, L>), vg, dim3(256), st, *p)
+    if (p->dtype == 1) { if (lph == 8) QV(__nv_bfloat16, 8); else if (lph == 16) QV(__nv_bfloat16, 16); else QV(__nv_bfloat16, 32); }
+    else { if (lph == 8) QV(float, 8); else if (lph == 16) QV(float, 16); else QV(float, 32); }
+#undef QV
+    return gb_launch_rc();
+  }
   const dim3 grid((unsigned)((items + 7) / 8));
   if (p->dtype == 1) GB_PDL_LAUNCH(ll_qkv_store_kernel<__nv_bfloat16>, grid, dim3(256), st, *p);
   else GB_PDL_LAUNCH(ll_qkv_store_kernel<float>, grid, dim3(256), st, *p);

@@ -1,12 +1,13 @@
 // Token-step matrix-vector products of layer-list models (contract in gb_layers.h).  One token is bound by weight bytes
 // and by the number of dependent launches, so what lies between two products (residual add with the norm of the
 // sublayer's output, gated group norm, final norm) is the prologue of the second one: every block makes the input
-// vector it needs in shared memory, and one block writes the new residual for the kernels after it.
+// vector it needs in shared memory, and one block writes the new residual for the kernels after it.  Weights do not depend
+// on the kernel before, so the first loads of a block's rows are issued ahead of the wait for it; a block walks several
+// rows when there are many, with the next row's loads issued before the current row is reduced.
 #include <type_traits>
 
 #include "sm100_common.cuh"
 #include "gb_layers.h"
-#include "decode_fmt.cuh"
 #include "layers_util.cuh"
 
 namespace gb {
@@ -44,24 +45,28 @@ struct LlGemv {
   const void* x16; long long ldx;
   const float* x; const float* y; long long ldy; const float* w1; const float* w2; float eps; float* x_out;
   const void* y16; long long ldy16; const void* z16; long long ldz; int parts;
+  const float* v32; const float* sq; int n_sq;
   void* out; long long ldo; int out_f32; float softcap;
 };
 
 // Input vector of sequence b into xs[0, K).
 template <int PRO, typename XT>
-__device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restrict__ xs, float* red) {
+__device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restrict__ xs, float* red, float* part_inv) {
   const int tid = threadIdx.x, d = a.d;
   if constexpr (PRO == 1) {
     const float* xr = a.x + (long long)b * d;
     constexpr int KEEP = 16;                       // values per thread kept in registers (d up to 4096)
     float v[KEEP];
+    const bool writes = blockIdx.x == 0 && a.x_out != nullptr;
     if (a.y) {
       const float* yr = a.y + b * a.ldy;
+      float xv[KEEP];
       float ss = 0.f;
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
         const int i = tid + k * LV_THREADS;
         v[k] = i < d ? yr[i] : 0.f;
+        xv[k] = i < d ? xr[i] : 0.f;
         ss += v[k] * v[k];
       }
       for (int i = tid + KEEP * LV_THREADS; i < d; i += LV_THREADS) ss += yr[i] * yr[i];
@@ -69,15 +74,12 @@ __device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restri
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
         const int i = tid + k * LV_THREADS;
-        if (i < d) v[k] = xr[i] + v[k] * inv * a.w1[i];
+        if (i < d) v[k] = xv[k] + v[k] * inv * a.w1[i];
       }
-      for (int i = tid; i < d; i += LV_THREADS) {
-        const int k = (i - tid) / LV_THREADS;
-        if (k >= KEEP) {
-          const float o = xr[i] + yr[i] * inv * a.w1[i];
-          if (blockIdx.x == 0 && a.x_out) a.x_out[(long long)b * d + i] = o;
-          if (!a.w2) xs[i] = Cvt<XT>::from_f(o);
-        }
+      for (int i = tid + KEEP * LV_THREADS; i < d; i += LV_THREADS) {
+        const float o = xr[i] + yr[i] * inv * a.w1[i];
+        if (writes) a.x_out[(long long)b * d + i] = o;
+        xs[i] = Cvt<XT>::from_f(o);
       }
     } else {
 #pragma unroll
@@ -86,11 +88,11 @@ __device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restri
         v[k] = i < d ? xr[i] : 0.f;
       }
       for (int i = tid + KEEP * LV_THREADS; i < d; i += LV_THREADS) {
-        if (blockIdx.x == 0 && a.x_out) a.x_out[(long long)b * d + i] = xr[i];
-        if (!a.w2) xs[i] = Cvt<XT>::from_f(xr[i]);
+        if (writes) a.x_out[(long long)b * d + i] = xr[i];
+        xs[i] = Cvt<XT>::from_f(xr[i]);
       }
     }
-    if (blockIdx.x == 0 && a.x_out) {
+    if (writes) {
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
         const int i = tid + k * LV_THREADS;
@@ -100,10 +102,7 @@ __device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restri
     if (a.w2) {                                    // the model's last norm on top (host: d <= KEEP * LV_THREADS)
       float ss = 0.f;
 #pragma unroll
-      for (int k = 0; k < KEEP; ++k) {
-        const int i = tid + k * LV_THREADS;
-        if (i < d) ss += v[k] * v[k];
-      }
+      for (int k = 0; k < KEEP; ++k) ss += v[k] * v[k];      // values past d are zero
       const float inv = ll_inv_rms(ll_block_sum(ss, red), d, a.eps);
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
@@ -116,6 +115,20 @@ __device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restri
       const int i = tid + k * LV_THREADS;
       if (i < d) xs[i] = Cvt<XT>::from_f(v[k]);
     }
+  } else if constexpr (PRO == 3) {                 // gated values and their sums of squares from the step kernel
+    const float* vr = a.v32 + (long long)b * d;
+    const float* sq = a.sq + (long long)b * a.n_sq;
+    const int per = d / a.parts, nq = a.n_sq / a.parts, warp = tid >> 5, lane = tid & 31;
+    for (int p = warp; p < a.parts; p += LV_WARPS) {
+      float ss = 0.f;
+      for (int i = lane; i < nq; i += 32) ss += sq[p * nq + i];
+      ss = warp_sum(ss);
+      if (lane == 0) part_inv[p] = ll_inv_rms(ss, per, a.eps);
+    }
+    __syncthreads();
+#pragma unroll 4
+    for (int i = tid; i < d; i += LV_THREADS) xs[i] = Cvt<XT>::from_f(vr[i] * part_inv[i / per] * a.w1[i]);
+    __syncthreads();                               // part_inv is the next sequence's, too
   } else {                                         // PRO == 2: gated norm in equal parts, one warp per part
     const XT* yr = reinterpret_cast<const XT*>(a.y16) + b * a.ldy16;
     const XT* zr = reinterpret_cast<const XT*>(a.z16) + b * a.ldz;
@@ -124,12 +137,12 @@ __device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restri
       for (int p = warp; p < a.parts; p += LV_WARPS) {
         float ss = 0.f;
         for (int i = lane; i < per; i += 32) {
-          const float v = Cvt<XT>::to_f(yr[p * per + i]) * ll_silu(Cvt<XT>::to_f(zr[p * per + i]));
+          const float v = Cvt<XT>::to_f(yr[p * per + i]) * ll_silu_t<XT>(Cvt<XT>::to_f(zr[p * per + i]));
           ss += v * v;
         }
         const float inv = ll_inv_rms(warp_sum(ss), per, a.eps);
         for (int i = lane; i < per; i += 32) {
-          const float v = Cvt<XT>::to_f(yr[p * per + i]) * ll_silu(Cvt<XT>::to_f(zr[p * per + i]));
+          const float v = Cvt<XT>::to_f(yr[p * per + i]) * ll_silu_t<XT>(Cvt<XT>::to_f(zr[p * per + i]));
           xs[p * per + i] = Cvt<XT>::from_f(v * inv * a.w1[p * per + i]);
         }
       }
@@ -141,11 +154,11 @@ __device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restri
 #pragma unroll
         for (int k = 0; k < KEEP; ++k) {
           const int i = tid + k * LV_THREADS;
-          v[k] = i < per ? Cvt<XT>::to_f(yr[p * per + i]) * ll_silu(Cvt<XT>::to_f(zr[p * per + i])) : 0.f;
+          v[k] = i < per ? Cvt<XT>::to_f(yr[p * per + i]) * ll_silu_t<XT>(Cvt<XT>::to_f(zr[p * per + i])) : 0.f;
           ss += v[k] * v[k];
         }
         for (int i = tid + KEEP * LV_THREADS; i < per; i += LV_THREADS) {
-          const float t = Cvt<XT>::to_f(yr[p * per + i]) * ll_silu(Cvt<XT>::to_f(zr[p * per + i]));
+          const float t = Cvt<XT>::to_f(yr[p * per + i]) * ll_silu_t<XT>(Cvt<XT>::to_f(zr[p * per + i]));
           ss += t * t;
         }
         const float inv = ll_inv_rms(ll_block_sum(ss, red), per, a.eps);
@@ -155,7 +168,7 @@ __device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restri
           if (i < per) xs[p * per + i] = Cvt<XT>::from_f(v[k] * inv * a.w1[p * per + i]);
         }
         for (int i = tid + KEEP * LV_THREADS; i < per; i += LV_THREADS) {
-          const float t = Cvt<XT>::to_f(yr[p * per + i]) * ll_silu(Cvt<XT>::to_f(zr[p * per + i]));
+          const float t = Cvt<XT>::to_f(yr[p * per + i]) * ll_silu_t<XT>(Cvt<XT>::to_f(zr[p * per + i]));
           xs[p * per + i] = Cvt<XT>::from_f(t * inv * a.w1[p * per + i]);
         }
       }
@@ -164,81 +177,130 @@ __device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restri
   for (int i = d + tid; i < a.K; i += LV_THREADS) xs[i] = Cvt<XT>::from_f(0.f);
 }
 
-template <int FMT, int NB, int KS, typename XT>
-__device__ __forceinline__ void ll_row(const uint8_t* __restrict__ wrow, int K, const XT* x, long long ldx, int nb, int ks,
-                                       float (&acc)[NB]) {
-  const int lane = threadIdx.x & 31;
-#pragma unroll 4
-  for (int u = lane + 32 * ks; u < (K >> 3); u += 32 * KS) {
-    float w[8];
-    load8<FMT>(wrow, u, w);
+// Raw stored values of one 8-value unit.
+template <int FMT> struct LlRaw;
+template <> struct LlRaw<GB_W_BF16> {
+  uint4 q;
+  __device__ __forceinline__ void load(const uint8_t* row, int u) { q = __ldg(reinterpret_cast<const uint4*>(row) + u); }
+  __device__ __forceinline__ void expand(float (&w)[8]) const {
+    const uint32_t v[4] = {q.x, q.y, q.z, q.w};
 #pragma unroll
-    for (int j = 0; j < NB; ++j)
-      if (j < nb) acc[j] += ll_dot8(w, x + j * ldx + 8 * u);
+    for (int i = 0; i < 4; ++i) { const float2 f = Cvt<__nv_bfloat16>::unpack2(v[i]); w[2 * i] = f.x; w[2 * i + 1] = f.y; }
   }
+};
+template <> struct LlRaw<GB_W_F32> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const uint8_t* row, int u) {
+    a = __ldg(reinterpret_cast<const float4*>(row) + 2 * u);
+    b = __ldg(reinterpret_cast<const float4*>(row) + 2 * u + 1);
+  }
+  __device__ __forceinline__ void expand(float (&w)[8]) const {
+    w[0] = a.x; w[1] = a.y; w[2] = a.z; w[3] = a.w; w[4] = b.x; w[5] = b.y; w[6] = b.z; w[7] = b.w;
+  }
+};
+
+template <int FMT, int NB, typename XT>
+__device__ __forceinline__ void ll_accum(const LlRaw<FMT>& raw, int u, const XT* x, long long ldx, int nb, float (&acc)[NB]) {
+  float w[8];
+  raw.expand(w);
+#pragma unroll
+  for (int j = 0; j < NB; ++j)
+    if (j < nb) acc[j] += ll_dot8(w, x + j * ldx + 8 * u);
 }
 
 // KS warps share a stored row (short rows spread over more of the machine); NB sequences per pass over the row.
 template <int FMT, typename XT, int PRO, int SWI, int NB, int KS>
 __global__ void __launch_bounds__(LV_THREADS) ll_gemv_kernel(const __grid_constant__ LlGemv a) {
-  pdl_wait();
+  constexpr int PF = (SWI ? 4 : 8) / (FMT == GB_W_F32 ? 2 : 1);      // units per lane and row that are loaded ahead
   extern __shared__ __align__(16) uint8_t lv_dyn[];
   __shared__ float red[LV_WARPS];
+  __shared__ float part_inv[PRO == 3 ? 256 : 1];
   __shared__ float part[2][LV_WARPS][NB];
   XT* xs = reinterpret_cast<XT*>(lv_dyn);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ric = warp / KS, ks = warp % KS;
+  const int n_out = SWI ? a.N / 2 : a.N, units = a.K >> 3, u0 = lane + 32 * ks;
+  constexpr int RPB = LV_WARPS / KS, US = 32 * KS;
+  auto row_of = [&](int j) { return a.W + (SWI ? (long long)(j >> 6) * 128 + (j & 63) : (long long)j) * a.row_bytes; };
+  LlRaw<FMT> g[PF], up[SWI ? PF : 1];
+  auto fetch = [&](int j) {
+    if (j >= n_out) return;
+    const uint8_t* w = row_of(j);
+#pragma unroll
+    for (int k = 0; k < PF; ++k)
+      if (u0 + k * US < units) {
+        g[k].load(w, u0 + k * US);
+        if constexpr (SWI != 0) up[k].load(w + 64 * a.row_bytes, u0 + k * US);
+      }
+  };
+  fetch(blockIdx.x * RPB + ric);
+  pdl_wait();
   const XT* xin = reinterpret_cast<const XT*>(a.x16);
   long long ldx = a.ldx;
   if constexpr (PRO != 0) {
-    for (int b = 0; b < a.B; ++b) ll_prologue<PRO, XT>(a, b, xs + (long long)b * a.K, red);
+    for (int b = 0; b < a.B; ++b) ll_prologue<PRO, XT>(a, b, xs + (long long)b * a.K, red, part_inv);
     __syncthreads();
     xin = xs;
     ldx = a.K;
   }
-  const int n_out = SWI ? a.N / 2 : a.N;
-  const int j = blockIdx.x * (LV_WARPS / KS) + ric;
-  const bool live = j < n_out;
-  const long long row = SWI ? (long long)(j >> 6) * 128 + (j & 63) : j;
-  const uint8_t* w0 = a.W + (live ? row : 0) * a.row_bytes;
-  const uint8_t* w1 = w0 + 64 * a.row_bytes;
-  for (int b0 = 0; b0 < a.B; b0 += NB) {
-    const int nb = min(NB, a.B - b0);
-    float acc[NB], acu[NB];
+  // every warp of the block makes the same number of trips: rows past the end still take part in the barriers
+  for (int j0 = blockIdx.x * RPB; j0 < n_out; j0 += gridDim.x * RPB) {
+    const int j = j0 + ric;
+    const bool live = j < n_out;
+    for (int b0 = 0; b0 < a.B; b0 += NB) {
+      const int nb = min(NB, a.B - b0);
+      float acc[NB], acu[NB];
 #pragma unroll
-    for (int k = 0; k < NB; ++k) { acc[k] = 0.f; acu[k] = 0.f; }
-    if (live) {
-      ll_row<FMT, NB, KS, XT>(w0, a.K, xin + b0 * ldx, ldx, nb, ks, acc);
-      if constexpr (SWI != 0) ll_row<FMT, NB, KS, XT>(w1, a.K, xin + b0 * ldx, ldx, nb, ks, acu);
-    }
+      for (int k = 0; k < NB; ++k) { acc[k] = 0.f; acu[k] = 0.f; }
+      if (live) {
+        if (b0 > 0) fetch(j);
+        const XT* xb = xin + b0 * ldx;
 #pragma unroll
-    for (int k = 0; k < NB; ++k) {
-      acc[k] = warp_sum(acc[k]);
-      if constexpr (SWI != 0) acu[k] = warp_sum(acu[k]);
-    }
-    if constexpr (KS > 1) {
-      if (lane == 0) {
-#pragma unroll
-        for (int k = 0; k < NB; ++k) { part[0][warp][k] = acc[k]; part[1][warp][k] = acu[k]; }
-      }
-      __syncthreads();
-      if (ks == 0) {
-#pragma unroll
-        for (int k = 0; k < NB; ++k) {
-          acc[k] = 0.f; acu[k] = 0.f;
-#pragma unroll
-          for (int s = 0; s < KS; ++s) { acc[k] += part[0][ric * KS + s][k]; acu[k] += part[1][ric * KS + s][k]; }
+        for (int k = 0; k < PF; ++k)
+          if (u0 + k * US < units) {
+            ll_accum<FMT, NB, XT>(g[k], u0 + k * US, xb, ldx, nb, acc);
+            if constexpr (SWI != 0) ll_accum<FMT, NB, XT>(up[k], u0 + k * US, xb, ldx, nb, acu);
+          }
+        const uint8_t* w = row_of(j);
+#pragma unroll 4
+        for (int u = u0 + PF * US; u < units; u += US) {
+          LlRaw<FMT> r0, r1;
+          r0.load(w, u);
+          if constexpr (SWI != 0) r1.load(w + 64 * a.row_bytes, u);
+          ll_accum<FMT, NB, XT>(r0, u, xb, ldx, nb, acc);
+          if constexpr (SWI != 0) ll_accum<FMT, NB, XT>(r1, u, xb, ldx, nb, acu);
         }
       }
-      __syncthreads();
-    }
-    if (live && ks == 0 && lane == 0) {
+      if (b0 + NB >= a.B) fetch(j + gridDim.x * RPB);
 #pragma unroll
       for (int k = 0; k < NB; ++k) {
-        if (k >= nb) continue;
-        float v = SWI ? ll_silu(acc[k]) * acu[k] : acc[k];
-        if (a.softcap > 0.f) v = a.softcap * tanhf(v / a.softcap);
-        if (a.out_f32) reinterpret_cast<float*>(a.out)[(long long)(b0 + k) * a.ldo + j] = v;
-        else reinterpret_cast<XT*>(a.out)[(long long)(b0 + k) * a.ldo + j] = Cvt<XT>::from_f(v);
+        acc[k] = warp_sum(acc[k]);
+        if constexpr (SWI != 0) acu[k] = warp_sum(acu[k]);
+      }
+      if constexpr (KS > 1) {
+        if (lane == 0) {
+#pragma unroll
+          for (int k = 0; k < NB; ++k) { part[0][warp][k] = acc[k]; part[1][warp][k] = acu[k]; }
+        }
+        __syncthreads();
+        if (ks == 0) {
+#pragma unroll
+          for (int k = 0; k < NB; ++k) {
+            acc[k] = 0.f; acu[k] = 0.f;
+#pragma unroll
+            for (int s = 0; s < KS; ++s) { acc[k] += part[0][ric * KS + s][k]; acu[k] += part[1][ric * KS + s][k]; }
+          }
+        }
+        __syncthreads();
+      }
+      if (live && ks == 0 && lane == 0) {
+#pragma unroll
+        for (int k = 0; k < NB; ++k) {
+          if (k >= nb) continue;
+          float v = SWI ? ll_silu(acc[k]) * acu[k] : acc[k];
+          if (a.softcap > 0.f) v = a.softcap * tanhf(v / a.softcap);
+          if (a.out_f32) reinterpret_cast<float*>(a.out)[(long long)(b0 + k) * a.ldo + j] = v;
+          else reinterpret_cast<XT*>(a.out)[(long long)(b0 + k) * a.ldo + j] = Cvt<XT>::from_f(v);
+        }
       }
     }
   }
@@ -249,11 +311,21 @@ static int ll_gemv_go(const LlGemv& a, cudaStream_t st) {
   const size_t smem = PRO ? (size_t)a.B * a.K * sizeof(XT) : 0;
   if (smem > 200 * 1024) return -3;
   const int n_out = SWI ? a.N / 2 : a.N;
-  const bool split = n_out <= 8192 && a.K >= 256;
-#define GO(NB, KS) GB_PDL_LAUNCH_SMEM((ll_gemv_kernel<FMT, XT, PRO, SWI, NB, KS>), dim3((n_out + LV_WARPS / KS - 1) / (LV_WARPS / KS)), \
-                                      dim3(LV_THREADS), smem, st, a)
-  if (a.B == 1) { if (split) GO(1, 4); else GO(1, 1); }
-  else { if (split) GO(4, 4); else GO(4, 1); }
+  // warps per row: enough of them to keep loads in flight on every SM
+  const int ks = n_out < 148 * 16 ? 4 : n_out < 148 * 64 ? 2 : 1;
+  // blocks: what is resident at once, and then so many that all of them make the same number of trips
+#define GO(NB, KS)                                                                                                                 \
+  do {                                                                                                                             \
+    auto kern = ll_gemv_kernel<FMT, XT, PRO, SWI, NB, KS>;                                                                         \
+    static int occ = 0;                                                                                                            \
+    if (!occ && (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&occ, kern, LV_THREADS, 16 * 1024) != cudaSuccess || occ < 1)) occ = 2; \
+    const int groups = (n_out + LV_WARPS / KS - 1) / (LV_WARPS / KS), trips = (groups + 148 * occ - 1) / (148 * occ);              \
+    GB_PDL_LAUNCH_SMEM(kern, dim3((groups + trips - 1) / trips), dim3(LV_THREADS), smem, st, a);                                   \
+  } while (0)
+#define GOK(NB) do { if (ks == 4) GO(NB, 4); else if (ks == 2) GO(NB, 2); else GO(NB, 1); } while (0)
+  if (a.B == 1) GOK(1);
+  else GOK(4);
+#undef GOK
 #undef GO
   return gb_launch_rc();
 }
@@ -264,6 +336,7 @@ static int ll_gemv_pro(const LlGemv& a, int prologue, int swiglu, cudaStream_t s
     case 0: return swiglu ? ll_gemv_go<FMT, XT, 0, 1>(a, st) : ll_gemv_go<FMT, XT, 0, 0>(a, st);
     case 1: return swiglu ? ll_gemv_go<FMT, XT, 1, 1>(a, st) : ll_gemv_go<FMT, XT, 1, 0>(a, st);
     case 2: return swiglu ? -1 : ll_gemv_go<FMT, XT, 2, 0>(a, st);
+    case 3: return swiglu ? -1 : ll_gemv_go<FMT, XT, 3, 0>(a, st);
   }
   return -1;
 }
@@ -279,7 +352,9 @@ extern "C" int gb_ll_gemv(const gb_ll_gemv_args* p, cudaStream_t st) {
   if (p->prologue == 0 && (!p->x16 || p->ldx % 8)) return -1;
   if (p->prologue == 1 && (!p->x || (p->y && !p->w1) || (p->w2 && p->d > 4096))) return -1;
   if (p->prologue == 2 && (!p->y16 || !p->z16 || !p->w1 || p->parts <= 0 || p->d % p->parts)) return -1;
+  if (p->prologue == 3 && (!p->v32 || !p->sq || !p->w1 || p->parts <= 0 || p->parts > 256 || p->d % p->parts || p->n_sq <= 0 || p->n_sq % p->parts)) return -1;
   LlGemv a{};
+  a.v32 = p->v32; a.sq = p->sq; a.n_sq = p->n_sq;
   a.W = static_cast<const uint8_t*>(p->W); a.row_bytes = rb; a.N = p->N; a.K = p->K; a.B = p->B; a.d = p->d;
   a.x16 = p->x16; a.ldx = p->ldx; a.x = p->x; a.y = p->y; a.ldy = p->ldy; a.w1 = p->w1; a.w2 = p->w2; a.eps = p->eps;
   a.x_out = p->x_out; a.y16 = p->y16; a.ldy16 = p->ldy16; a.z16 = p->z16; a.ldz = p->ldz; a.parts = p->parts;

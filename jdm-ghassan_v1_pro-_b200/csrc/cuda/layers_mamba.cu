@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(128) ll_conv_kernel(const __grid_constant__ gb
     float s = bias + w[0] * cur;
 #pragma unroll
     for (int k = 1; k < MAXT; ++k) s += w[k] * x[k - 1];
-    ll_conv_out<T>(a, (long long)b * a.n + t, c, ll_silu(s));
+    ll_conv_out<T>(a, (long long)b * a.n + t, c, ll_silu_t<T>(s));
 #pragma unroll
     for (int k = MAXT - 1; k > 0; --k) x[k] = x[k - 1];
     x[0] = cur;
@@ -67,6 +67,84 @@ __global__ void __launch_bounds__(128) ll_conv_kernel(const __grid_constant__ gb
   // The block of the first tile is the only reader of this channel's carried inputs, so it also replaces them.
   if (t0 == 0)
     for (int t = max(0, a.n - a.taps); t < a.n; ++t) ring[(long long)((p0 + t) % a.taps) * C + c] = proj[t * a.ld_proj + c];
+}
+
+// Eight channels per thread (sizes and pitches in multiples of eight), `tile` tokens: one 16-byte load and store per token,
+// the inputs of the last taps - 1 tokens in registers.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) ll_conv_vec_kernel(const __grid_constant__ gb_ll_mamba_args a, int tile) {
+  pdl_wait();
+  const int n = a.H * a.P, gn = a.G * a.N, C = n + 2 * gn;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 8, b = blockIdx.z, t0 = blockIdx.y * tile;
+  if (c >= C) return;
+  const int p0 = a.st[b].abs_pos;
+  const T* src = reinterpret_cast<const T*>(a.proj) + (long long)b * a.n * a.ld_proj + n + c;
+  T* ring = reinterpret_cast<T*>(a.conv_state) + (long long)b * TAPS * C + c;
+  float w[TAPS][8], x[TAPS][8], bias[8];     // x[k]: inputs k + 1 tokens before the current one
+  ll_load8(a.conv_b + c, bias);
+  {
+    float f[TAPS][8];                        // the taps of eight channels are consecutive
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) ll_load8(a.conv_w + (long long)c * TAPS + 8 * i, f[i]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e)
+#pragma unroll
+      for (int k = 0; k < TAPS; ++k) { const int i = e * TAPS + TAPS - 1 - k; w[k][e] = f[i >> 3][i & 7]; }
+  }
+#pragma unroll
+  for (int k = 1; k < TAPS; ++k) {
+    const int t = t0 - k;
+    if (t >= 0) ll_load8(src + t * a.ld_proj, x[k - 1]);
+    else if (p0 + t >= 0) ll_load8(ring + (long long)((p0 + t) % TAPS) * C, x[k - 1]);
+    else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[k - 1][e] = 0.f;
+    }
+  }
+  T* dst;
+  long long step;
+  if (c < n) {
+    const int h = c / a.P;
+    dst = reinterpret_cast<T*>(a.xh) + (long long)h * a.Pp + (c - h * a.P);
+    step = (long long)a.H * a.Pp;
+  } else {
+    const bool is_b = c < n + gn;
+    const int e = c - n - (is_b ? 0 : gn), g = e / a.N;
+    dst = reinterpret_cast<T*>(is_b ? a.bc : a.cc) + (long long)g * a.Np + (e - g * a.N);
+    step = (long long)a.G * a.Np;
+  }
+  dst += ((long long)b * a.n + t0) * step;
+  const int t1 = min(a.n, t0 + tile);
+  constexpr int PF = 4;
+  for (int t = t0; t < t1; t += PF) {
+    float in[PF][8];
+#pragma unroll
+    for (int u = 0; u < PF; ++u)
+      if (t + u < t1) ll_load8(src + (t + u) * a.ld_proj, in[u]);
+#pragma unroll
+    for (int u = 0; u < PF; ++u) {
+      if (t + u >= t1) break;
+      float o[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        float s = bias[e] + w[0][e] * in[u][e];
+#pragma unroll
+        for (int k = 1; k < TAPS; ++k) s += w[k][e] * x[k - 1][e];
+        o[e] = ll_silu_t<T>(s);
+#pragma unroll
+        for (int k = TAPS - 1; k > 0; --k) x[k][e] = x[k - 1][e];
+        x[0][e] = in[u][e];
+      }
+      ll_store8(dst, o);
+      dst += step;
+    }
+  }
+  if (t0 == 0)                             // this block alone read the carried inputs of these channels
+    for (int t = max(0, a.n - TAPS); t < a.n; ++t) {
+      float v[8];
+      ll_load8(src + t * a.ld_proj, v);
+      ll_store8(ring + (long long)((p0 + t) % TAPS) * C, v);
+    }
 }
 
 // ---------------------------------------------------------------------------------------------- recurrence
@@ -194,7 +272,7 @@ __global__ void __launch_bounds__(256) ll_mamba_step_kernel(const __grid_constan
       float s = a.conv_b[c] + a.conv_w[(long long)c * a.taps + a.taps - 1] * Cvt<T>::to_f(cur);
       for (int k = 1; k < a.taps; ++k)
         if (pos - k >= 0) s += a.conv_w[(long long)c * a.taps + a.taps - 1 - k] * Cvt<T>::to_f(ring[(long long)((pos - k) % a.taps) * C + c]);
-      v = Cvt<T>::to_f(Cvt<T>::from_f(ll_silu(s)));
+      v = Cvt<T>::to_f(Cvt<T>::from_f(ll_silu_t<T>(s)));
       if (i < 32 || owner) ring[(long long)(pos % a.taps) * C + c] = cur;
     }
     if (i < 32) sX[i] = v;
@@ -205,10 +283,27 @@ __global__ void __launch_bounds__(256) ll_mamba_step_kernel(const __grid_constan
   const float decay = expf(-expf(a.A_log[h]) * dt);
   __syncthreads();
   const float x = sX[pr];
-  const float y = ll_sum8(S.step(decay, dt * x, sB, sC, slice));
-  if (live) {
-    S.store(srow, a.Ns, slice);
-    if (slice == 0) reinterpret_cast<T*>(a.y)[b * a.ld_y + h * a.P + p] = Cvt<T>::from_f(y + a.D[h] * x);
+  const float y = ll_sum8(S.step(decay, dt * x, sB, sC, slice)) + a.D[h] * x;
+  if (live) S.store(srow, a.Ns, slice);
+  if (a.gated == nullptr) {
+    if (live && slice == 0) reinterpret_cast<T*>(a.y)[b * a.ld_y + h * a.P + p] = Cvt<T>::from_f(y);
+    return;
+  }
+  // y silu(z) for the norm that follows, and this block's part of its sum of squares
+  __shared__ float s_sq[8];
+  float v = 0.f;
+  if (live && slice == 0) {
+    v = Cvt<T>::to_f(Cvt<T>::from_f(y)) * ll_silu_t<T>(Cvt<T>::to_f(row[h * a.P + p]));
+    a.gated[(long long)b * n + h * a.P + p] = v;
+  }
+  v = warp_sum(v * v);
+  if ((tid & 31) == 0) s_sq[tid >> 5] = v;
+  __syncthreads();
+  if (tid == 0) {
+    float q = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) q += s_sq[w];
+    a.gated_sq[((long long)b * a.H + h) * gridDim.x + blockIdx.x] = q;
   }
 }
 
@@ -230,11 +325,11 @@ __global__ void __launch_bounds__(128) ll_gated_norm_kernel(const __grid_constan
 #pragma unroll
   for (int k = 0; k < KEEP; ++k) {
     const int i = tid + 128 * k;
-    v[k] = i < per ? Cvt<T>::to_f(y[i]) * ll_silu(Cvt<T>::to_f(z[i])) : 0.f;
+    v[k] = i < per ? Cvt<T>::to_f(y[i]) * ll_silu_t<T>(Cvt<T>::to_f(z[i])) : 0.f;
     ss += v[k] * v[k];
   }
   for (int i = tid + 128 * KEEP; i < per; i += 128) {
-    const float u = Cvt<T>::to_f(y[i]) * ll_silu(Cvt<T>::to_f(z[i]));
+    const float u = Cvt<T>::to_f(y[i]) * ll_silu_t<T>(Cvt<T>::to_f(z[i]));
     ss += u * u;
   }
   ss = warp_sum(ss);
@@ -247,7 +342,57 @@ __global__ void __launch_bounds__(128) ll_gated_norm_kernel(const __grid_constan
     if (i < per) o[i] = Cvt<T>::from_f(v[k] * inv * a.norm_w[c0 + i]);
   }
   for (int i = tid + 128 * KEEP; i < per; i += 128)
-    o[i] = Cvt<T>::from_f(Cvt<T>::to_f(y[i]) * ll_silu(Cvt<T>::to_f(z[i])) * inv * a.norm_w[c0 + i]);
+    o[i] = Cvt<T>::from_f(Cvt<T>::to_f(y[i]) * ll_silu_t<T>(Cvt<T>::to_f(z[i])) * inv * a.norm_w[c0 + i]);
+}
+
+// The same with 16-byte accesses: VPT vectors of eight values per thread.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(256) ll_gated_norm_vec_kernel(const __grid_constant__ gb_ll_mamba_args a) {
+  pdl_wait();
+  __shared__ float red[8];
+  const int per = a.H * a.P / a.norm_groups, tid = threadIdx.x, nv = per >> 3;
+  const long long r = blockIdx.x;
+  const int c0 = blockIdx.y * per;
+  const T* y = reinterpret_cast<const T*>(a.y) + r * a.ld_y + c0;
+  const T* z = reinterpret_cast<const T*>(a.proj) + r * a.ld_proj + c0;
+  T* o = reinterpret_cast<T*>(a.out) + r * a.ld_out + c0;
+  float v[VPT][8], zz[VPT][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = tid + blockDim.x * k;
+    if (i < nv) { ll_load8(y + 8 * i, v[k]); ll_load8(z + 8 * i, zz[k]); }
+  }
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    if (tid + blockDim.x * k >= nv) break;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) { v[k][e] *= ll_silu_t<T>(zz[k][e]); ss += v[k][e] * v[k][e]; }
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) tot += red[w];
+  const float inv = ll_inv_rms(tot, per, a.eps);
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = tid + blockDim.x * k;
+    if (i >= nv) break;
+    float g[8];
+    ll_load8(a.norm_w + c0 + 8 * i, g);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[k][e] *= inv * g[e];
+    ll_store8(o + 8 * i, v[k]);
+  }
+}
+
+static bool ll_vec_ok(const gb_ll_mamba_args& a) {
+  return a.P % 8 == 0 && a.N % 8 == 0 && a.Pp % 8 == 0 && a.Np % 8 == 0 && a.ld_proj % 8 == 0 && a.ld_y % 8 == 0 && a.ld_out % 8 == 0 &&
+         ((reinterpret_cast<uintptr_t>(a.proj) | reinterpret_cast<uintptr_t>(a.xh) | reinterpret_cast<uintptr_t>(a.bc) |
+           reinterpret_cast<uintptr_t>(a.cc) | reinterpret_cast<uintptr_t>(a.conv_state) | reinterpret_cast<uintptr_t>(a.y) |
+           reinterpret_cast<uintptr_t>(a.out) | reinterpret_cast<uintptr_t>(a.norm_w) | reinterpret_cast<uintptr_t>(a.conv_w) |
+           reinterpret_cast<uintptr_t>(a.conv_b)) & 15) == 0;
 }
 
 template <typename T>
@@ -265,6 +410,17 @@ static int ll_scan_go(const gb_ll_mamba_args& a, bool step, cudaStream_t st) {
 template <typename T>
 static int ll_conv_go(const gb_ll_mamba_args& a, cudaStream_t st) {
   const int C = a.H * a.P + 2 * a.G * a.N;
+  // tokens per thread: long enough to pay for loading the taps, short enough to fill the machine
+  const long long groups = (long long)((C / 8 + 127) / 128) * a.B;
+  int tile = 64;
+  while (tile > 8 && groups * ((a.n + tile - 1) / tile) < 148 * 4) tile >>= 1;
+  if (ll_vec_ok(a) && a.taps >= 2 && a.taps <= 4 && (a.n + tile - 1) / tile <= 65535) {
+    const dim3 vg((C / 8 + 127) / 128, (a.n + tile - 1) / tile, a.B);
+    if (a.taps == 2) GB_PDL_LAUNCH((ll_conv_vec_kernel<T, 2>), vg, dim3(128), st, a, tile);
+    else if (a.taps == 3) GB_PDL_LAUNCH((ll_conv_vec_kernel<T, 3>), vg, dim3(128), st, a, tile);
+    else GB_PDL_LAUNCH((ll_conv_vec_kernel<T, 4>), vg, dim3(128), st, a, tile);
+    return gb_launch_rc();
+  }
   const dim3 grid((C + 127) / 128, (a.n + CONV_TT - 1) / CONV_TT, a.B);
   if (a.taps <= 4) GB_PDL_LAUNCH((ll_conv_kernel<T, 4>), grid, dim3(128), st, a);
   else if (a.taps <= 8) GB_PDL_LAUNCH((ll_conv_kernel<T, 8>), grid, dim3(128), st, a);
@@ -298,6 +454,7 @@ extern "C" int gb_ll_scan(const gb_ll_mamba_args* p, cudaStream_t st) {
 extern "C" int gb_ll_mamba_step(const gb_ll_mamba_args* p, cudaStream_t st) {
   if (const int rc = ll_mamba_check(p)) return rc;
   if (p->n != 1) return -3;
+  if (p->gated && !p->gated_sq) return -1;
   return p->dtype == 1 ? ll_scan_go<__nv_bfloat16>(*p, true, st) : ll_scan_go<float>(*p, true, st);
 }
 
@@ -305,6 +462,17 @@ extern "C" int gb_ll_gated_norm(const gb_ll_mamba_args* p, cudaStream_t st) {
   if (const int rc = ll_mamba_check(p)) return rc;
   if (!p->out || !p->norm_w || p->norm_groups <= 0 || (p->H * p->P) % p->norm_groups) return -1;
   const dim3 grid(p->B * p->n, p->norm_groups);
+  const int per = p->H * p->P / p->norm_groups;
+  if (per % 8 == 0 && per <= 8192 && ll_vec_ok(*p)) {
+    const int nv = per / 8, threads = nv >= 256 ? 256 : (nv + 31) / 32 * 32, vpt = (nv + threads - 1) / threads;
+#define GN(T, V) GB_PDL_LAUNCH((ll_gated_norm_vec_kernel<T, V>), grid, dim3(threads), st, *p)
+#define GNT(T) do { if (vpt == 1) GN(T, 1); else if (vpt == 2) GN(T, 2); else if (vpt == 3) GN(T, 3); else GN(T, 4); } while (0)
+    if (p->dtype == 1) GNT(__nv_bfloat16);
+    else GNT(float);
+#undef GNT
+#undef GN
+    return gb_launch_rc();
+  }
   if (p->dtype == 1) GB_PDL_LAUNCH(ll_gated_norm_kernel<__nv_bfloat16>, grid, dim3(128), st, *p);
   else GB_PDL_LAUNCH(ll_gated_norm_kernel<float>, grid, dim3(128), st, *p);
   return gb_launch_rc();

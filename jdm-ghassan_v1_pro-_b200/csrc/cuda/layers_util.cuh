@@ -7,6 +7,37 @@ namespace gb {
 __device__ __forceinline__ float ll_inv_rms(float sum_sq, int n, float eps) { return 1.0f / sqrtf(sum_sq / (float)n + eps); }
 __device__ __forceinline__ float ll_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float ll_silu(float z) { return z / (1.0f + expf(-z)); }
+// The same for results that are rounded to 16 bits: hardware exponential and reciprocal (relative error about 2^-21).
+__device__ __forceinline__ float ll_sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(fminf(-z, 80.f))); }
+template <typename T> __device__ __forceinline__ float ll_sigmoid_t(float z) {
+  if constexpr (sizeof(T) == 4) return ll_sigmoid(z);
+  else return ll_sigmoid_fast(z);
+}
+template <typename T> __device__ __forceinline__ float ll_silu_t(float z) {
+  if constexpr (sizeof(T) == 4) return ll_silu(z);
+  else return z * ll_sigmoid_fast(z);
+}
+// eight consecutive values
+__device__ __forceinline__ void ll_load8(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 q = *reinterpret_cast<const uint4*>(p);
+  const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { const float2 f = Cvt<__nv_bfloat16>::unpack2(w[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
+}
+__device__ __forceinline__ void ll_load8(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void ll_store8(__nv_bfloat16* p, const float (&v)[8]) {
+  uint4 q;
+  q.x = Cvt<__nv_bfloat16>::pack2(v[0], v[1]); q.y = Cvt<__nv_bfloat16>::pack2(v[2], v[3]);
+  q.z = Cvt<__nv_bfloat16>::pack2(v[4], v[5]); q.w = Cvt<__nv_bfloat16>::pack2(v[6], v[7]);
+  *reinterpret_cast<uint4*>(p) = q;
+}
+__device__ __forceinline__ void ll_store8(float* p, const float (&v)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
 // log(1 + e^z), without overflow for large z
 __device__ __forceinline__ float ll_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 

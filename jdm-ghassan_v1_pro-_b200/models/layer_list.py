@@ -275,24 +275,25 @@ def random_parameters(cfg: LayerListConfig, seed: int = 0, dtype=None, device="c
     """Random tensors of the right shapes and sane scales (benchmarks and demonstrations): matrices ~ N(0, 1/in), norms
     around one, decays between slow and fast."""
     import torch
-    g = torch.Generator(device="cpu").manual_seed(seed)
+    g = torch.Generator(device=device).manual_seed(seed)
+    kw = dict(generator=g, device=device)
     dtype = dtype or torch.bfloat16
     out = {}
     for n, shape in cfg.tensor_shapes().items():
         leaf = n.split(".")[-1] if not n.endswith("conv.b") else "conv.b"
         if leaf in ("norm1", "norm2", "norm"):
-            t = 1.0 + 0.1 * torch.randn(shape, generator=g)
+            t = 1.0 + 0.1 * torch.randn(shape, **kw)
         elif leaf == "A_log":
-            t = torch.log(torch.empty(shape).uniform_(0.5, 8.0, generator=g))
+            t = torch.log(torch.empty(shape, device=device).uniform_(0.5, 8.0, generator=g))
         elif leaf == "dt_bias":
-            t = torch.empty(shape).uniform_(-5.0, -1.0, generator=g)
+            t = torch.empty(shape, device=device).uniform_(-5.0, -1.0, generator=g)
         elif leaf in ("D", "sink"):
-            t = torch.randn(shape, generator=g)
+            t = torch.randn(shape, **kw)
         elif leaf == "conv.b":
-            t = 0.1 * torch.randn(shape, generator=g)
+            t = 0.1 * torch.randn(shape, **kw)
         elif leaf == "embed":
-            t = torch.randn(shape, generator=g)
+            t = torch.randn(shape, **kw)
         else:
-            t = torch.randn(shape, generator=g) * shape[-1] ** -0.5
-        out[n] = t.to(dtype).to(device)
+            t = torch.randn(shape, **kw) * shape[-1] ** -0.5
+        out[n] = t.to(dtype)
     return out

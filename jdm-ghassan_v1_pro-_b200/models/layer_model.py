@@ -152,7 +152,16 @@ class LayerModel:
         return act
 
     # ------------------------------------------------------------------ mixer arguments
-    def attn_args(self, i: int, cache, st, slot: int, B: int, n: int, pos0_max: int) -> K.AttnArgs:
+    def _cs(self, freq):
+        return self.buf("cs%d" % freq.data_ptr(), 2 * freq.numel(), torch.float32)
+
+    def _rotations(self, st, B: int, n: int):
+        """Cosines and sines of this pass's rows, once per distinct rotation of the model."""
+        for f in {t.data_ptr(): t for t in self.freq if t is not None}.values():
+            K.rotations(f, st, B, n, self._cs(f))
+            self.launches += 1
+
+    def attn_args(self, i: int, cache, st, slot: int, B: int, n: int, pos0_max: int, rotations: bool = False) -> K.AttnArgs:
         m: AttentionMixer = self.cfg.layers[i].mixer
         w = self.weights[i]
         a = K.AttnArgs()
@@ -161,6 +170,7 @@ class LayerModel:
         f = self.freq[i]
         if f is not None:
             a.rot_dims, a.rot_half, a.freq = m.rot.dims, int(m.rot.half), f.data_ptr()
+            a.cs = self._cs(f).data_ptr() if rotations else None
         a.qk_norm, a.eps, a.scale = int(m.qk_norm), self.cfg.eps, m.scale
         a.window, a.keep, a.cap = m.window, cache.keep, cache.cap
         proj = self.buf("proj", _up(w.w_in.shape[0], 8))
@@ -209,7 +219,7 @@ class LayerModel:
         w = self.weights[i]
         self._gemm(self.x16, w.w_in, self.buf("proj", _up(w.w_in.shape[0], 8)), B * n)
         if isinstance(self.cfg.layers[i].mixer, AttentionMixer):
-            a = self.attn_args(i, cache, st, slot, B, n, pos0_max)
+            a = self.attn_args(i, cache, st, slot, B, n, pos0_max, True)
             K.qkv_store(a)
             if n == 1:
                 K.attn_decode(a)
@@ -247,6 +257,7 @@ class LayerModel:
         x = self.x[0]
         K.embed(ids, self.embed, x, self.x16, d)
         self.launches += 1
+        self._rotations(st, B, n)
         for i, spec in enumerate(cfg.layers):
             w = self.weights[i]
             mixed = self._mix_rows(i, mem.layers[i], st, slot, B, n, pos0)
@@ -297,6 +308,7 @@ class LayerModel:
         x, other = self.x
         K.embed(ids, self.embed, x, self.x16, d)
         self.launches += 1
+        self._rotations(st, B, 1)
         y = [self.buf("tok_y%d" % k, _up(d, 4), torch.float32, rows=K.GEMV_MAX_BATCH) for k in range(2)]
         pend = None                       # norm weight of a sublayer output in y[0] that is not yet in the residual
 
@@ -318,7 +330,7 @@ class LayerModel:
             w, m, c = self.weights[i], spec.mixer, mem.layers[i]
             from_x(w.w_in, self.buf("proj", _up(w.w_in.shape[0], 8)))
             if isinstance(m, AttentionMixer):
-                a = self.attn_args(i, c, st, slot, B, 1, -1)
+                a = self.attn_args(i, c, st, slot, B, 1, -1, True)
                 K.qkv_store(a)
                 K.attn_decode(a)
                 self.launches += 3
@@ -326,10 +338,20 @@ class LayerModel:
                 to_y(w.w_o, w.norm1, prologue=0, d=m.out_features, x16=mixed, ldx=mixed.stride(0))
             else:
                 a = self.mamba_args(i, c, st, slot, B, 1)
-                K.mamba_step(a)
+                if m.heads % m.norm_groups == 0 and m.norm_groups <= 256:
+                    # the step leaves y silu(z) and sums of squares that add up to the norm's groups
+                    tiles = (m.vdim + 31) // 32
+                    gated = self.buf("gated", m.out_features, torch.float32, rows=K.GEMV_MAX_BATCH)
+                    sq = self.buf("gated_sq", m.heads * tiles, torch.float32, rows=K.GEMV_MAX_BATCH)
+                    a.gated, a.gated_sq = gated.data_ptr(), sq.data_ptr()
+                    K.mamba_step(a)
+                    to_y(w.w_o, w.norm1, prologue=3, d=m.out_features, v32=gated, sq=sq, n_sq=m.heads * tiles, w1=w.vec["norm"],
+                         parts=m.norm_groups)
+                else:
+                    K.mamba_step(a)
+                    to_y(w.w_o, w.norm1, prologue=2, d=m.out_features, y16=a.y, ldy16=a.ld_y, z16=a.proj, ldz=a.ld_proj,
+                         w1=w.vec["norm"], parts=m.norm_groups)
                 self.launches += 1
-                to_y(w.w_o, w.norm1, prologue=2, d=m.out_features, y16=a.y, ldy16=a.ld_y, z16=a.proj, ldz=a.ld_proj, w1=w.vec["norm"],
-                     parts=m.norm_groups)
             if spec.mlp is not None:
                 act = self.buf("act", w.w_gu.shape[0] // 2)
                 from_x(w.w_gu, act, swiglu=1)

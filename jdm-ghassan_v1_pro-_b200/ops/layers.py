@@ -23,6 +23,7 @@ class GemvArgs(ctypes.Structure):
         ("x16", c_vp), ("ldx", c_ll),
         ("x", c_vp), ("y", c_vp), ("ldy", c_ll), ("w1", c_vp), ("w2", c_vp), ("eps", c_float), ("x_out", c_vp),
         ("y16", c_vp), ("ldy16", c_ll), ("z16", c_vp), ("ldz", c_ll), ("parts", c_int),
+        ("v32", c_vp), ("sq", c_vp), ("n_sq", c_int),
         ("out", c_vp), ("ldo", c_ll), ("out_f32", c_int), ("softcap", c_float),
     ]
 
@@ -31,7 +32,7 @@ class AttnArgs(ctypes.Structure):
     _fields_ = [
         ("dtype", c_int), ("B", c_int), ("n", c_int), ("H", c_int), ("G", c_int),
         ("dk", c_int), ("dv", c_int), ("dkp", c_int), ("dvp", c_int),
-        ("rot_dims", c_int), ("rot_half", c_int), ("freq", c_vp), ("qk_norm", c_int), ("eps", c_float), ("scale", c_float),
+        ("rot_dims", c_int), ("rot_half", c_int), ("freq", c_vp), ("cs", c_vp), ("qk_norm", c_int), ("eps", c_float), ("scale", c_float),
         ("window", c_int), ("keep", c_int), ("cap", c_int),
         ("proj", c_vp), ("ld_proj", c_ll), ("gate", c_int), ("sink", c_vp),
         ("q", c_vp), ("cache_k", c_vp), ("cache_v", c_vp), ("out", c_vp), ("ldo", c_ll),
@@ -47,7 +48,8 @@ class MambaArgs(ctypes.Structure):
         ("conv_w", c_vp), ("conv_b", c_vp), ("dt_bias", c_vp), ("A_log", c_vp), ("D", c_vp),
         ("norm_w", c_vp), ("norm_groups", c_int), ("eps", c_float),
         ("conv_state", c_vp), ("ssm", c_vp), ("xh", c_vp), ("bc", c_vp), ("cc", c_vp),
-        ("y", c_vp), ("ld_y", c_ll), ("out", c_vp), ("ld_out", c_ll), ("st", c_vp), ("chunk_ws", c_vp), ("status", c_vp),
+        ("y", c_vp), ("ld_y", c_ll), ("out", c_vp), ("ld_out", c_ll), ("gated", c_vp), ("gated_sq", c_vp),
+        ("st", c_vp), ("chunk_ws", c_vp), ("status", c_vp),
     ]
 
 
@@ -95,6 +97,11 @@ def advance(state, pos_out, n):
 
 def gemv(a: GemvArgs):
     _call("gb_ll_gemv", ctypes.byref(a))
+
+
+def rotations(freq, state, B, n, cs):
+    """Cosines and sines of ``n`` consecutive positions of each sequence: ``cs`` [B * n, pairs, 2]."""
+    _call("gb_ll_rotations", _p(freq), c_int(freq.numel()), _p(state), c_int(B), c_int(n), _p(cs))
 
 
 def qkv_store(a: AttnArgs):

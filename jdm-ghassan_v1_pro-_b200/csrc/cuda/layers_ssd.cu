@@ -9,10 +9,12 @@
 // first sum, the scaled x of the state update, S_prev itself) it enters as two bf16 terms, value and remainder, so that
 // products keep 16 bits of it, and the state accumulates in fp32.
 //
-// One CTA per (sequence, head, run of chunks): warps 0-3 own the chunk's token rows (weights of the first sum, outputs),
-// warps 4-7 the state rows and the scaled x, warp 8 loads tiles with TMA, warp 9 issues the MMAs, warp 10 turns raw step
-// sizes into dt and L one chunk ahead.  When there are fewer heads than SMs the tokens are cut into segments: a first
-// launch computes what every segment adds to the state from zero, the second starts each segment from the combination.
+// One CTA per (sequence, head, run of chunks): warps 0-7 own the chunk's token rows (weights of the first sum, outputs;
+// warps w and w + 4 share 32 rows and take alternate 32-column blocks), warps 8-11 the state rows and the scaled x, warp 12
+// loads tiles with TMA, warp 13 issues the MMAs, warp 14 turns raw step sizes into dt and L one chunk ahead.  The state
+// chain (S_prev -> operand, scaled x, state update) runs ahead of the output chain.  When there are fewer heads than SMs
+// the tokens are cut into segments: a first launch computes what every segment adds to the state from zero, a small
+// kernel turns those into the state before each segment, the last launch starts from there.
 #include <algorithm>
 
 #include "sm100_common.cuh"
@@ -24,7 +26,8 @@ namespace gb {
 
 constexpr int SD_Q = 128;                  // tokens per chunk
 constexpr int SD_N = 128;                  // padded state size
-constexpr int SD_THREADS = 352;
+constexpr int SD_W_STATE = 8, SD_W_TMA = 12, SD_W_MMA = 13, SD_W_DT = 14;
+constexpr int SD_THREADS = 480;
 
 struct SsdParams {
   int B, n, H, P, N, G, Ns;
@@ -34,7 +37,8 @@ struct SsdParams {
   __nv_bfloat16* y; long long ld_y;
   const gb_seq_state* st;
   int n_chunks, seg_chunks, n_seg, state_only;
-  float* ws_state;                         // [B, H, n_seg, P, Ns]: slot 0 = state before the call, slot k + 1 = segment k's part
+  float* ws_state;                         // [B, H, n_seg, P, Ns]: slot k = state before segment k (first launch: slot 0 as it
+                                           // is, slot k + 1 = what segment k adds from zero)
   float* ws_decay;                         // [B, H, n_seg]: log2 decay over segment k
   int* status;
 };
@@ -59,8 +63,10 @@ struct SsdCfg {
   static constexpr uint32_t TBC = SD_Q * SD_N * 2, TX = SD_Q * PP * 2, STAGE = 2 * TBC + TX;
   static constexpr uint32_t TS = SD_N * PP * 2;
   static constexpr size_t TILES = (size_t)STAGES * STAGE + 2 * TS + 2 * TX;
-  static constexpr size_t SMEM = TILES + 2 * 2 * SD_Q * 4 + 192;
-  static constexpr int COL_Y = 128 * NG, COL_Y2 = COL_Y + PP, COL_S = COL_Y2 + PP;
+  static constexpr size_t SMEM = TILES + 2 * (2 * SD_Q + 96) * 4 + 128;
+  // the products with both terms of S_prev side by side (one pass over C) where tensor memory has the columns
+  static constexpr int NY2 = PP == 64 ? 2 : 1;
+  static constexpr int COL_Y = 128 * NG, COL_Y2 = COL_Y + PP, COL_S = COL_Y2 + PP * NY2;
 };
 
 template <int PP>
@@ -81,7 +87,8 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
   uint8_t* sXlo = sXhi + K::TX;
   float* sL = reinterpret_cast<float*>(sXlo + K::TX);       // [2][128] L in log2 units
   float* sV = sL + 2 * SD_Q;                                // [2][128] log2(dt) - L
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * SD_Q);
+  float* sU = sV + 2 * SD_Q;                                // [2][96] dt exp(L_end - L), L_end = L at the end of the token's 32-block
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sU + 2 * 96);
   uint64_t* full = bars;               // 2
   uint64_t* empty = bars + 2;          // 2
   uint64_t* l_full = bars + 4;         // 2
@@ -105,21 +112,21 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
   if (threadIdx.x == 0) {
     for (int s = 0; s < 2; ++s) {
       mbar_init(&full[s], 1);
-      mbar_init(&empty[s], so ? 1 : 5);
+      mbar_init(&empty[s], so ? 1 : 9);
       mbar_init(&l_full[s], 1);
-      mbar_init(&l_empty[s], so ? 4 : 8);
+      mbar_init(&l_empty[s], so ? 4 : 12);
     }
     mbar_init(g_full, 1);
-    mbar_init(m_ready, 4);
+    mbar_init(m_ready, 8);
     mbar_init(y_full, 1);
-    mbar_init(y_empty, 4);
+    mbar_init(y_empty, 8);
     mbar_init(s_ready, 4);
     mbar_init(xw_ready, 4);
     mbar_init(s_full, 1);
     *abort_flag = 0;
     fence_barrier_init();
   }
-  if (warp == 9) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
+  if (warp == SD_W_MMA) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -127,7 +134,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
   const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
 #define SD_WAIT(bar, ph, code) if (!at_wait(bar, ph, p.status, code, abort_flag)) break
 
-  if (warp == 8) {
+  if (warp == SD_W_TMA) {
     // ------------------------------------------------------------------ TMA
     if (lane == 0) {
       for (int c = 0; c < nc; ++c) {
@@ -142,15 +149,25 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       }
     }
     __syncwarp();
-  } else if (warp == 9) {
+  } else if (warp == SD_W_MMA) {
     // ------------------------------------------------------------------ MMA
     if (lane == 0) {
       const uint32_t id_g = make_idesc_f16(1, 0, 0, SD_Q, SD_Q);
       const uint32_t id_y = make_idesc_f16(1, 0, 1, SD_Q, PP);
+      const uint32_t id_y2 = make_idesc_f16(1, 0, 1, SD_Q, PP * K::NY2);
       const uint32_t id_s = make_idesc_f16(1, 1, 1, SD_N, PP);
+      // Descriptors advance by address alone (units of 16 bytes): a tile of 128 rows has panels of 1024 units, a step of 16
+      // along K is 2 units inside a K-major panel and 128 units (16 rows) in an MN-major one.
+      const uint64_t d_st = make_smem_desc_sw128(smem_u32(smem), 16, 1024), d_mn = make_smem_desc_sw128(smem_u32(smem), SD_Q * 128, 1024);
+      const uint64_t d_s = make_smem_desc_sw128(smem_u32(sShi), SD_N * 128, 1024), d_xw = make_smem_desc_sw128(smem_u32(sXhi), SD_Q * 128, 1024);
       auto scores = [&](int c) {
-        const uint32_t st = smem_u32(smem + (c % K::STAGES) * K::STAGE);
-        mma_kmajor_kmajor<SD_N>(tm + (c % K::NG) * 128, st, st + K::TBC, id_g, false);
+        const uint64_t dc = d_st + (c % K::STAGES) * (K::STAGE >> 4);
+        const uint32_t to = tm + (c % K::NG) * 128;
+#pragma unroll
+        for (int kk = 0; kk < SD_N / 16; ++kk) {
+          const uint32_t off = (kk >> 2) * 1024 + (kk & 3) * 2;
+          umma_f16(to, dc + off, dc + (K::TBC >> 4) + off, id_g, kk ? 1u : 0u);
+        }
         umma_commit(g_full);
       };
       bool ok = true;
@@ -160,29 +177,17 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       }
       for (int c = 0; c < nc && ok; ++c) {
         const int s = c % K::STAGES;
-        const uint32_t st = smem_u32(smem + s * K::STAGE), sx = st + 2 * K::TBC;
+        const uint64_t dc = d_st + s * (K::STAGE >> 4), dmn = d_mn + s * (K::STAGE >> 4);
         if (so) SD_WAIT(&full[s], (c / K::STAGES) & 1, ST_TIMEOUT_FULL);
         SD_WAIT(s_ready, c & 1, ST_TIMEOUT_EMPTY);
         if (!so) {
           if (c > 0) SD_WAIT(y_empty, (c - 1) & 1, ST_TIMEOUT_TMEM_EMPTY);
           tc_fence_after();
-          mma_kmajor_mnmajor<SD_N>(tm + K::COL_Y2, st, smem_u32(sShi), id_y, false);
-          mma_kmajor_mnmajor<SD_N>(tm + K::COL_Y2, st, smem_u32(sSlo), id_y, true);
-          SD_WAIT(m_ready, c & 1, ST_TIMEOUT_TMEM_EMPTY);
-          tc_fence_after();
-          const uint32_t m0 = tm + (c % K::NG) * 128;
 #pragma unroll
-          for (int part = 0; part < 2; ++part)
+          for (int part = 0; part < 2 / K::NY2; ++part)
 #pragma unroll
-            for (int kk = 0; kk < SD_Q / 16; ++kk)
-              umma_f16_ts(tm + K::COL_Y, m0 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8,
-                          make_smem_desc_sw128(sx + kk * 2048, SD_Q * 128, 1024), id_y, (part || kk) ? 1u : 0u);
-          umma_commit(y_full);
-          if (K::STAGES == 2 && c + 1 < nc) {
-            SD_WAIT(&full[(c + 1) % K::STAGES], ((c + 1) / K::STAGES) & 1, ST_TIMEOUT_FULL);
-            tc_fence_after();
-            scores(c + 1);
-          }
+            for (int kk = 0; kk < SD_N / 16; ++kk)
+              umma_f16(tm + K::COL_Y2, dc + (kk >> 2) * 1024 + (kk & 3) * 2, d_s + part * (K::TS >> 4) + kk * 128, id_y2, (part || kk) ? 1u : 0u);
         }
         SD_WAIT(xw_ready, c & 1, ST_TIMEOUT_EMPTY);
         tc_fence_after();
@@ -190,20 +195,31 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
         for (int part = 0; part < 2; ++part)
 #pragma unroll
           for (int kk = 0; kk < SD_Q / 16; ++kk)
-            umma_f16(tm + K::COL_S, make_smem_desc_sw128(st + K::TBC + kk * 2048, SD_Q * 128, 1024),
-                     make_smem_desc_sw128(smem_u32(part ? sXlo : sXhi) + kk * 2048, SD_Q * 128, 1024), id_s, 1u);
+            umma_f16(tm + K::COL_S, dmn + (K::TBC >> 4) + kk * 128, d_xw + part * (K::TX >> 4) + kk * 128, id_s, 1u);
         umma_commit(s_full);
+        if (!so) {
+          SD_WAIT(m_ready, c & 1, ST_TIMEOUT_TMEM_EMPTY);
+          tc_fence_after();
+          const uint32_t m0 = tm + (c % K::NG) * 128;
+#pragma unroll
+          for (int part = 0; part < 2; ++part)
+#pragma unroll
+            for (int kk = 0; kk < SD_Q / 16; ++kk)
+              umma_f16_ts(tm + K::COL_Y, m0 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8, dmn + (2 * K::TBC >> 4) + kk * 128, id_y,
+                          (part || kk) ? 1u : 0u);
+          umma_commit(y_full);
+        }
         umma_commit(&empty[s]);
-        if (!so && K::STAGES == 1 && c + 1 < nc) {
-          SD_WAIT(y_full, c & 1, ST_TIMEOUT_TMEM_FULL);      // the one score buffer still holds this chunk's weights
-          SD_WAIT(&full[0], (c + 1) & 1, ST_TIMEOUT_FULL);
+        if (!so && c + 1 < nc) {
+          if (K::NG == 1) SD_WAIT(y_full, c & 1, ST_TIMEOUT_TMEM_FULL);      // the one score buffer still holds this chunk's weights
+          SD_WAIT(&full[(c + 1) % K::STAGES], ((c + 1) / K::STAGES) & 1, ST_TIMEOUT_FULL);
           tc_fence_after();
           scores(c + 1);
         }
       }
     }
     __syncwarp();
-  } else if (warp == 10) {
+  } else if (warp == SD_W_DT) {
     // ------------------------------------------------------------------ dt and L
     const float bias = p.dt_bias[h], na2 = -expf(p.A_log[h]) * 1.4426950408889634f;
     for (int c = 0; c < nc; ++c) {
@@ -222,54 +238,66 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
         if (lane >= o) inc += v;
       }
       const float before = inc - run;
+      // L at the end of this lane's 32-token block
+      const float Lb = __shfl_sync(0xffffffffu, before + cum[3], lane | 7);
       SD_WAIT(&l_empty[s], ((c >> 1) & 1) ^ 1, ST_TIMEOUT_EMPTY);
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         const float L = before + cum[k];
         sL[s * SD_Q + lane * 4 + k] = L;
         sV[s * SD_Q + lane * 4 + k] = log2f(dt[k]) - L;
+        if (lane < 24) sU[s * 96 + lane * 4 + k] = dt[k] * sd_ex2(Lb - L);
       }
       __syncwarp();
       if (lane == 0) mbar_arrive(&l_full[s]);
     }
     __syncwarp();
-  } else if (warp < 4) {
+  } else if (warp < SD_W_STATE) {
     // ------------------------------------------------------------------ token rows
-    const int r = threadIdx.x;
+    const int quarter = warp & 3, half = warp >> 2, r = quarter * 32 + lane;
     const float D = p.D[h];
     for (int c = 0; c < nc && !so; ++c) {
       const int ls = c & 1, s = c % K::STAGES, t = (c_lo + c) * SD_Q + r;
       SD_WAIT(&l_full[ls], (c >> 1) & 1, ST_TIMEOUT_FULL);
-      const float L = sL[ls * SD_Q + r];
-      const float4* v4 = reinterpret_cast<const float4*>(sV + ls * SD_Q);
+      const float* Lrow = sL + ls * SD_Q;
+      const float L = Lrow[r];
       const uint32_t tg = tm + (c % K::NG) * 128 + lane_base;
       SD_WAIT(g_full, c & 1, ST_TIMEOUT_TMEM_FULL);
       tc_fence_after();
       // weights (C_t . B_s) exp(L_t - L_s) dt_s, written over the scores they come from: per 32 columns, 16 columns of
-      // packed values and 16 of packed remainders
-#pragma unroll 1
-      for (int q = 0; q < 4; ++q) {
+      // packed values and 16 of packed remainders.  Left of the diagonal block the exponential is a product of a factor
+      // of the row and one of the column, both against the L at the end of the column's block (neither exceeds 1).
+#pragma unroll
+      for (int q0 = 0; q0 < 4; q0 += 2) {
+        const int q = q0 + half;
         uint32_t hi[16], lo[16];
-        if (q <= warp) {
+        if (q < quarter) {
           uint32_t rg[32];
           tmem_ld_32x32(tg + q * 32, rg);
+          const float f = sd_ex2(L - Lrow[q * 32 + 31]);
+          const float4* u4 = reinterpret_cast<const float4*>(sU + ls * 96) + q * 8;
           tmem_ld_wait();
 #pragma unroll
           for (int k = 0; k < 8; ++k) {
-            const float4 v = v4[q * 8 + k];
-            float m[4];
-            m[0] = __uint_as_float(rg[4 * k]) * sd_ex2(fminf(L + v.x, 126.f));
-            m[1] = __uint_as_float(rg[4 * k + 1]) * sd_ex2(fminf(L + v.y, 126.f));
-            m[2] = __uint_as_float(rg[4 * k + 2]) * sd_ex2(fminf(L + v.z, 126.f));
-            m[3] = __uint_as_float(rg[4 * k + 3]) * sd_ex2(fminf(L + v.w, 126.f));
-            if (q == warp) {
+            const float4 u = u4[k];
+            sd_split2(__uint_as_float(rg[4 * k]) * (f * u.x), __uint_as_float(rg[4 * k + 1]) * (f * u.y), hi[2 * k], lo[2 * k]);
+            sd_split2(__uint_as_float(rg[4 * k + 2]) * (f * u.z), __uint_as_float(rg[4 * k + 3]) * (f * u.w), hi[2 * k + 1], lo[2 * k + 1]);
+          }
+        } else if (q == quarter) {
+          uint32_t rg[32];
+          tmem_ld_32x32(tg + q * 32, rg);
+          const float4* v4 = reinterpret_cast<const float4*>(sV + ls * SD_Q) + q * 8;
+          tmem_ld_wait();
 #pragma unroll
-              for (int e = 0; e < 4; ++e)
-                if (4 * k + e > lane) m[e] = 0.f;
-            }
+          for (int k = 0; k < 8; ++k) {
+            const float4 v = v4[k];
+            float m[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) m[e] = 4 * k + e > lane ? 0.f : __uint_as_float(rg[4 * k + e]) * sd_ex2(L + m[e]);
             sd_split2(m[0], m[1], hi[2 * k], lo[2 * k]);
             sd_split2(m[2], m[3], hi[2 * k + 1], lo[2 * k + 1]);
           }
+          __syncwarp();
         } else {
 #pragma unroll
           for (int k = 0; k < 16; ++k) { hi[k] = 0u; lo[k] = 0u; }
@@ -282,22 +310,31 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(m_ready);
       const float eL = sd_ex2(L);
-      SD_WAIT(y_full, c & 1, ST_TIMEOUT_TMEM_FULL);
-      SD_WAIT(&full[s], (c / K::STAGES) & 1, ST_TIMEOUT_FULL);      // long since true; this thread reads x itself
-      tc_fence_after();
       const uint8_t* sx = smem + s * K::STAGE + 2 * K::TBC;
       T* yp = p.y + ((long long)b * p.n + t) * p.ld_y + h * p.P;
       const bool live = t < p.n;
       const bool vec = p.P == PP && ((reinterpret_cast<uintptr_t>(p.y) | (uintptr_t)(p.ld_y * 2)) & 15) == 0;
+      SD_WAIT(y_full, c & 1, ST_TIMEOUT_TMEM_FULL);
+      SD_WAIT(&full[s], (c / K::STAGES) & 1, ST_TIMEOUT_FULL);      // long since true; this thread reads x itself
+      tc_fence_after();
 #pragma unroll
-      for (int q = 0; q < PP / 32; ++q) {
+      for (int q0 = 0; q0 < PP / 64; ++q0) {
+        const int c0 = half * (PP / 2) + q0 * 32;
         uint32_t a[32], e[32];
-        tmem_ld_32x32(tm + K::COL_Y + lane_base + q * 32, a);
-        tmem_ld_32x32(tm + K::COL_Y2 + lane_base + q * 32, e);
-        tmem_ld_wait();
+        tmem_ld_32x32(tm + K::COL_Y + lane_base + c0, a);
+        tmem_ld_32x32(tm + K::COL_Y2 + lane_base + c0, e);
+        if constexpr (K::NY2 == 2) {
+          uint32_t e2[32];
+          tmem_ld_32x32(tm + K::COL_Y2 + PP + lane_base + c0, e2);
+          tmem_ld_wait();
+#pragma unroll
+          for (int k = 0; k < 32; ++k) e[k] = __float_as_uint(__uint_as_float(e[k]) + __uint_as_float(e2[k]));
+        } else {
+          tmem_ld_wait();
+        }
 #pragma unroll
         for (int k = 0; k < 4 && live; ++k) {
-          const int col = q * 32 + 8 * k;
+          const int col = c0 + 8 * k;
           const uint4 xq = *reinterpret_cast<const uint4*>(sx + (col >> 6) * (SD_Q * 128) + sw128_off(r, col & 63));
           const uint32_t xw[4] = {xq.x, xq.y, xq.z, xq.w};
           float v[8];
@@ -318,7 +355,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
               if (col + j < p.P) yp[col + j] = Cvt<T>::from_f(v[j]);
           }
         }
-        __syncwarp();                       // the next tensor-memory load is the whole warp's
+        __syncwarp();                       // the next tensor-memory access is the whole warp's
       }
       tc_fence_before();
       __syncwarp();
@@ -326,7 +363,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
     }
   } else {
     // ------------------------------------------------------------------ state rows and scaled x
-    const int r = threadIdx.x - 128;            // state column (0 .. 127) / token of the chunk
+    const int r = threadIdx.x - SD_W_STATE * 32;   // state column (0 .. 127) / token of the chunk
     const bool live_n = r < p.N;
     const long long per = (long long)p.P * p.Ns;
     float* home = p.ssm + bh * per;
@@ -334,62 +371,58 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
     const uint32_t ts = tm + K::COL_S + lane_base;
     const bool fresh = p.st[b].abs_pos == 0;
     // the state this run starts from
-#pragma unroll 1
+    const float* from = so || (p.n_seg == 1 && fresh) ? nullptr : p.n_seg == 1 ? home : ws + seg * per;
+#pragma unroll
     for (int q = 0; q < PP / 16; ++q) {
       uint32_t v[16];
 #pragma unroll
       for (int k = 0; k < 16; ++k) {
         const int pp = q * 16 + k;
-        float x = 0.f;
-        if (live_n && pp < p.P) {
-          const long long at = (long long)pp * p.Ns + r;
-          if (so) {
-            if (seg == 0) ws[at] = fresh ? 0.f : home[at];          // the second launch's last segment replaces `home`
-          } else if (p.n_seg == 1) {
-            x = fresh ? 0.f : home[at];
-          } else {
-            x = ws[at];
-            for (int j = 0; j < seg; ++j) x = x * sd_ex2(p.ws_decay[(long long)bh * p.n_seg + j]) + ws[(j + 1) * per + at];
-          }
-        }
-        v[k] = __float_as_uint(x);
+        v[k] = (from && live_n && pp < p.P) ? __float_as_uint(from[(long long)pp * p.Ns + r]) : 0u;
       }
       __syncwarp();
       tmem_st_32x16(ts + q * 16, v);
     }
     tmem_st_wait();
+    if (so && seg == 0 && live_n)                       // the last launch's last segment replaces `home`
+      for (int pp = 0; pp < p.P; ++pp) ws[(long long)pp * p.Ns + r] = fresh ? 0.f : home[(long long)pp * p.Ns + r];
     float total = 0.f;
     bool ok = true;
     for (int c = 0; c < nc; ++c) {
       const int ls = c & 1, s = c % K::STAGES;
       ok = false;
       SD_WAIT(&l_full[ls], (c >> 1) & 1, ST_TIMEOUT_FULL);
-      const float Ll = sL[ls * SD_Q + SD_Q - 1], dec = sd_ex2(Ll), w = sd_ex2(fminf(Ll + sV[ls * SD_Q + r], 126.f));
+      const float Ll = sL[ls * SD_Q + SD_Q - 1], dec = sd_ex2(Ll), w = sd_ex2(Ll + sV[ls * SD_Q + r]);
       total += Ll;
       if (c > 0) SD_WAIT(s_full, (c - 1) & 1, ST_TIMEOUT_TMEM_FULL);
       tc_fence_after();
 #pragma unroll
-      for (int q = 0; q < PP / 16; ++q) {
-        uint32_t v[16];
-        tmem_ld_32x16(ts + q * 16, v);
+      for (int q = 0; q < PP / 32; ++q) {
+        uint32_t v[32];
+        tmem_ld_32x32(ts + q * 32, v);
         tmem_ld_wait();
         if (!so) {
 #pragma unroll
-          for (int k = 0; k < 2; ++k) {
+          for (int k = 0; k < 4; ++k) {
             uint4 hi, lo;
             sd_split2(__uint_as_float(v[8 * k]), __uint_as_float(v[8 * k + 1]), hi.x, lo.x);
             sd_split2(__uint_as_float(v[8 * k + 2]), __uint_as_float(v[8 * k + 3]), hi.y, lo.y);
             sd_split2(__uint_as_float(v[8 * k + 4]), __uint_as_float(v[8 * k + 5]), hi.z, lo.z);
             sd_split2(__uint_as_float(v[8 * k + 6]), __uint_as_float(v[8 * k + 7]), hi.w, lo.w);
-            const int col = q * 16 + 8 * k;
+            const int col = q * 32 + 8 * k;
             const uint32_t off = (col >> 6) * (SD_N * 128) + sw128_off(r, col & 63);
             *reinterpret_cast<uint4*>(sShi + off) = hi;
             *reinterpret_cast<uint4*>(sSlo + off) = lo;
           }
         }
+        uint32_t w0[16], w1[16];
 #pragma unroll
-        for (int k = 0; k < 16; ++k) v[k] = __float_as_uint(__uint_as_float(v[k]) * dec);
-        tmem_st_32x16(ts + q * 16, v);
+        for (int k = 0; k < 16; ++k) {
+          w0[k] = __float_as_uint(__uint_as_float(v[k]) * dec);
+          w1[k] = __float_as_uint(__uint_as_float(v[16 + k]) * dec);
+        }
+        tmem_st_32x16(ts + q * 32, w0);
+        tmem_st_32x16(ts + q * 32 + 16, w1);
       }
       tmem_st_wait();
       tc_fence_before();
@@ -442,19 +475,34 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
     for (int k = 0; k < 64; ++k) __nanosleep(1000);
     __syncthreads();
   }
-  if (warp == 9) { tc_fence_after(); tmem_dealloc(tm, 512); }
+  if (warp == SD_W_MMA) { tc_fence_after(); tmem_dealloc(tm, 512); }
+}
+
+// ws slots 1 .. n_seg - 1 from "what segment k adds" to "state before the segment"; one thread per state value.
+__global__ void __launch_bounds__(256) ll_ssd_combine_kernel(float* __restrict__ ws, const float* __restrict__ decay, int n_seg, long long per) {
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i >= per) return;
+  float* w = ws + (long long)blockIdx.y * n_seg * per + i;
+  const float* d = decay + (long long)blockIdx.y * n_seg;
+  float s = w[0];
+#pragma unroll 4
+  for (int k = 1; k < n_seg; ++k) {
+    s = s * sd_ex2(d[k - 1]) + w[k * per];
+    w[k * per] = s;
+  }
 }
 
 struct SsdPlan { int n_chunks, seg_chunks, n_seg; };
 
-// Segments per head: the cheapest number of rounds over the SMs, where cutting at all costs the extra state pass.
+// Segments per head: the cheapest number of rounds over the SMs.  A CTA costs about three chunks to start and drain; a
+// state-only chunk about 0.7 of a full one.
 static SsdPlan ssd_plan(int BH, int n, int sms) {
   SsdPlan best{(n + SD_Q - 1) / SD_Q, 0, 1};
   best.seg_chunks = best.n_chunks;
-  double cost = (double)((BH + sms - 1) / sms) * best.n_chunks;
+  double cost = (double)((BH + sms - 1) / sms) * (best.n_chunks + 3.0);
   for (int s = 2; s <= 16 && s <= best.n_chunks; ++s) {
     const int per = (best.n_chunks + s - 1) / s, k = (best.n_chunks + per - 1) / per;
-    const double c = per * ((double)((BH * k + sms - 1) / sms) + 0.5 * ((BH * (k - 1) + sms - 1) / sms)) + 3.0;
+    const double c = (per + 3.0) * ((BH * k + sms - 1) / sms) + (0.7 * per + 3.0) * ((BH * (k - 1) + sms - 1) / sms) + 3.0;
     if (c < cost * 0.95) { cost = c; best.seg_chunks = per; best.n_seg = k; }
   }
   return best;
@@ -505,6 +553,8 @@ static int ssd_go(const gb_ll_mamba_args& a, int force_segments, cudaStream_t st
     p.state_only = 1;
     ll_ssd_kernel<PP><<<(unsigned)(BH * (plan.n_seg - 1)), SD_THREADS, K::SMEM, st>>>(tx, tb, tc, p);
     p.state_only = 0;
+    const long long per = (long long)a.P * a.Ns;
+    ll_ssd_combine_kernel<<<dim3((unsigned)((per + 255) / 256), (unsigned)BH), 256, 0, st>>>(p.ws_state, p.ws_decay, plan.n_seg, per);
   }
   ll_ssd_kernel<PP><<<(unsigned)(BH * plan.n_seg), SD_THREADS, K::SMEM, st>>>(tx, tb, tc, p);
   return gb_launch_rc();

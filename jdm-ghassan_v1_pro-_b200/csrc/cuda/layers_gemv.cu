@@ -311,8 +311,9 @@ static int ll_gemv_go(const LlGemv& a, cudaStream_t st) {
   const size_t smem = PRO ? (size_t)a.B * a.K * sizeof(XT) : 0;
   if (smem > 200 * 1024) return -3;
   const int n_out = SWI ? a.N / 2 : a.N;
-  // warps per row: enough of them to keep loads in flight on every SM
-  const int ks = n_out < 148 * 16 ? 4 : n_out < 148 * 64 ? 2 : 1;
+  // warps per row: enough of them to keep loads in flight on every SM, more for long rows
+  const int units = a.K >> 3;
+  const int ks = (n_out < 148 * 16 || units > 512) ? 4 : (n_out < 148 * 64 || units > 256) ? 2 : 1;
   // blocks: what is resident at once, and then so many that all of them make the same number of trips
 #define GO(NB, KS)                                                                                                                 \
   do {                                                                                                                             \

@@ -69,36 +69,43 @@ __global__ void __launch_bounds__(128) ll_conv_kernel(const __grid_constant__ gb
     for (int t = max(0, a.n - a.taps); t < a.n; ++t) ring[(long long)((p0 + t) % a.taps) * C + c] = proj[t * a.ld_proj + c];
 }
 
-// Eight channels per thread (sizes and pitches in multiples of eight), `tile` tokens: one 16-byte load and store per token,
-// the inputs of the last taps - 1 tokens in registers.
+// Four channels per thread (sizes and pitches in multiples of four), `tile` tokens: one vector load and store per token, the
+// inputs of the last taps - 1 tokens in registers, four tokens' loads ahead of their use.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) ll_conv_vec_kernel(const __grid_constant__ gb_ll_mamba_args a, int tile) {
   pdl_wait();
   const int n = a.H * a.P, gn = a.G * a.N, C = n + 2 * gn;
-  const int c = (blockIdx.x * 128 + threadIdx.x) * 8, b = blockIdx.z, t0 = blockIdx.y * tile;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 4, b = blockIdx.z, t0 = blockIdx.y * tile, t1 = min(a.n, t0 + tile);
   if (c >= C) return;
-  const int p0 = a.st[b].abs_pos;
+  constexpr int PF = 4;
   const T* src = reinterpret_cast<const T*>(a.proj) + (long long)b * a.n * a.ld_proj + n + c;
+  LlRaw4<T> in[PF];
+#pragma unroll
+  for (int u = 0; u < PF; ++u)
+    if (t0 + u < t1) in[u].load(src + (t0 + u) * a.ld_proj);
+  const int p0 = a.st[b].abs_pos;
   T* ring = reinterpret_cast<T*>(a.conv_state) + (long long)b * TAPS * C + c;
-  float w[TAPS][8], x[TAPS][8], bias[8];     // x[k]: inputs k + 1 tokens before the current one
-  ll_load8(a.conv_b + c, bias);
+  float w[TAPS][4], x[TAPS][4], bias[4];     // x[k]: inputs k + 1 tokens before the current one
+#pragma unroll
+  for (int e = 0; e < 4; ++e) bias[e] = a.conv_b[c + e];
   {
-    float f[TAPS][8];                        // the taps of eight channels are consecutive
+    float f[TAPS][4];                        // the taps of four channels are consecutive
 #pragma unroll
-    for (int i = 0; i < TAPS; ++i) ll_load8(a.conv_w + (long long)c * TAPS + 8 * i, f[i]);
+    for (int i = 0; i < TAPS; ++i) { LlRaw4<float> r; r.load(a.conv_w + (long long)c * TAPS + 4 * i); r.expand(f[i]); }
 #pragma unroll
-    for (int e = 0; e < 8; ++e)
+    for (int e = 0; e < 4; ++e)
 #pragma unroll
-      for (int k = 0; k < TAPS; ++k) { const int i = e * TAPS + TAPS - 1 - k; w[k][e] = f[i >> 3][i & 7]; }
+      for (int k = 0; k < TAPS; ++k) { const int i = e * TAPS + TAPS - 1 - k; w[k][e] = f[i >> 2][i & 3]; }
   }
 #pragma unroll
   for (int k = 1; k < TAPS; ++k) {
     const int t = t0 - k;
-    if (t >= 0) ll_load8(src + t * a.ld_proj, x[k - 1]);
-    else if (p0 + t >= 0) ll_load8(ring + (long long)((p0 + t) % TAPS) * C, x[k - 1]);
+    LlRaw4<T> r;
+    if (t >= 0) { r.load(src + t * a.ld_proj); r.expand(x[k - 1]); }
+    else if (p0 + t >= 0) { r.load(ring + (long long)((p0 + t) % TAPS) * C); r.expand(x[k - 1]); }
     else {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[k - 1][e] = 0.f;
+      for (int e = 0; e < 4; ++e) x[k - 1][e] = 0.f;
     }
   }
   T* dst;
@@ -114,36 +121,39 @@ __global__ void __launch_bounds__(128) ll_conv_vec_kernel(const __grid_constant_
     step = (long long)a.G * a.Np;
   }
   dst += ((long long)b * a.n + t0) * step;
-  const int t1 = min(a.n, t0 + tile);
-  constexpr int PF = 4;
   for (int t = t0; t < t1; t += PF) {
-    float in[PF][8];
+    LlRaw4<T> nx[PF];
 #pragma unroll
     for (int u = 0; u < PF; ++u)
-      if (t + u < t1) ll_load8(src + (t + u) * a.ld_proj, in[u]);
+      if (t + PF + u < t1) nx[u].load(src + (t + PF + u) * a.ld_proj);
 #pragma unroll
     for (int u = 0; u < PF; ++u) {
-      if (t + u >= t1) break;
-      float o[8];
+      if (t + u < t1) {
+        float cur[4];
+        in[u].expand(cur);
+        float4 o;
+        float* op = reinterpret_cast<float*>(&o);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        float s = bias[e] + w[0][e] * in[u][e];
+        for (int e = 0; e < 4; ++e) {
+          float s = bias[e] + w[0][e] * cur[e];
 #pragma unroll
-        for (int k = 1; k < TAPS; ++k) s += w[k][e] * x[k - 1][e];
-        o[e] = ll_silu_t<T>(s);
+          for (int k = 1; k < TAPS; ++k) s += w[k][e] * x[k - 1][e];
+          op[e] = ll_silu_t<T>(s);
 #pragma unroll
-        for (int k = TAPS - 1; k > 0; --k) x[k][e] = x[k - 1][e];
-        x[0][e] = in[u][e];
+          for (int k = TAPS - 1; k > 0; --k) x[k][e] = x[k - 1][e];
+          x[0][e] = cur[e];
+        }
+        ll_store4(dst, o);
+        dst += step;
       }
-      ll_store8(dst, o);
-      dst += step;
+      in[u] = nx[u];
     }
   }
   if (t0 == 0)                             // this block alone read the carried inputs of these channels
     for (int t = max(0, a.n - TAPS); t < a.n; ++t) {
-      float v[8];
-      ll_load8(src + t * a.ld_proj, v);
-      ll_store8(ring + (long long)((p0 + t) % TAPS) * C, v);
+      LlRaw4<T> r;
+      r.load(src + t * a.ld_proj);
+      r.store(ring + (long long)((p0 + t) % TAPS) * C);
     }
 }
 
@@ -411,11 +421,11 @@ template <typename T>
 static int ll_conv_go(const gb_ll_mamba_args& a, cudaStream_t st) {
   const int C = a.H * a.P + 2 * a.G * a.N;
   // tokens per thread: long enough to pay for loading the taps, short enough to fill the machine
-  const long long groups = (long long)((C / 8 + 127) / 128) * a.B;
+  const long long groups = (long long)((C / 4 + 127) / 128) * a.B;
   int tile = 64;
-  while (tile > 8 && groups * ((a.n + tile - 1) / tile) < 148 * 4) tile >>= 1;
+  while (tile > 8 && groups * ((a.n + tile - 1) / tile) < 148 * 6) tile >>= 1;
   if (ll_vec_ok(a) && a.taps >= 2 && a.taps <= 4 && (a.n + tile - 1) / tile <= 65535) {
-    const dim3 vg((C / 8 + 127) / 128, (a.n + tile - 1) / tile, a.B);
+    const dim3 vg((C / 4 + 127) / 128, (a.n + tile - 1) / tile, a.B);
     if (a.taps == 2) GB_PDL_LAUNCH((ll_conv_vec_kernel<T, 2>), vg, dim3(128), st, a, tile);
     else if (a.taps == 3) GB_PDL_LAUNCH((ll_conv_vec_kernel<T, 3>), vg, dim3(128), st, a, tile);
     else GB_PDL_LAUNCH((ll_conv_vec_kernel<T, 4>), vg, dim3(128), st, a, tile);

@@ -41,6 +41,23 @@ __device__ __forceinline__ void ll_store8(float* p, const float (&v)[8]) {
 // log(1 + e^z), without overflow for large z
 __device__ __forceinline__ float ll_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
+// four consecutive values, raw and expanded
+template <typename T> struct LlRaw4;
+template <> struct LlRaw4<__nv_bfloat16> {
+  uint2 q;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { q = *reinterpret_cast<const uint2*>(p); }
+  __device__ __forceinline__ void expand(float (&v)[4]) const {
+    const float2 a = Cvt<__nv_bfloat16>::unpack2(q.x), b = Cvt<__nv_bfloat16>::unpack2(q.y);
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+  }
+  __device__ __forceinline__ void store(__nv_bfloat16* p) const { *reinterpret_cast<uint2*>(p) = q; }
+};
+template <> struct LlRaw4<float> {
+  float4 q;
+  __device__ __forceinline__ void load(const float* p) { q = *reinterpret_cast<const float4*>(p); }
+  __device__ __forceinline__ void expand(float (&v)[4]) const { v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+  __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<float4*>(p) = q; }
+};
 __device__ __forceinline__ void ll_store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
 __device__ __forceinline__ void ll_store4(__nv_bfloat16* p, const float4& v) {
   uint2 q;

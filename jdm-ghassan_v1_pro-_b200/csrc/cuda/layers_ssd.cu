@@ -49,6 +49,39 @@ __device__ __forceinline__ float sd_ex2(float x) {
   return r;
 }
 
+// MMA and commit for a warp that runs converged: every lane passes the same operands, the lane with `on` != 0 issues.  The
+// operands then stay in uniform registers, which is where the instruction wants them; issued from a one-lane branch, each
+// MMA first moved its descriptors there and cost 70 to 100 cycles of issue time.
+__device__ __forceinline__ void sd_mma(uint32_t on, uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "setp.ne.b32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+      :
+      : "r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate), "r"(on)
+      : "memory");
+}
+__device__ __forceinline__ void sd_mma_ts(uint32_t on, uint32_t d, uint32_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "setp.ne.b32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+      :
+      : "r"(d), "r"(a), "l"(b), "r"(idesc), "r"(accumulate), "r"(on)
+      : "memory");
+}
+__device__ __forceinline__ void sd_commit(uint32_t on, uint64_t* bar) {
+  asm volatile(
+      "{\n\t.reg .pred q;\n\t"
+      "setp.ne.b32 q, %1, 0;\n\t"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
+      :
+      : "r"(smem_u32(bar)), "r"(on)
+      : "memory");
+}
+
 // 2 values -> packed bf16 pair and the packed remainders
 __device__ __forceinline__ void sd_split2(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = Cvt<__nv_bfloat16>::pack2(a, b);
@@ -130,7 +163,9 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tm = *tmem_slot;
+  // all 512 columns are this CTA's, so the allocation starts at column 0 (checked: addresses below are constants)
+  constexpr uint32_t tm = 0;
+  if (*tmem_slot != 0 && threadIdx.x == 0) { atomicCAS(p.status, 0, ST_BAD_ARGUMENT); *abort_flag = 1; }
   const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
 #define SD_WAIT(bar, ph, code) if (!at_wait(bar, ph, p.status, code, abort_flag)) break
 
@@ -151,7 +186,8 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
     __syncwarp();
   } else if (warp == SD_W_MMA) {
     // ------------------------------------------------------------------ MMA
-    if (lane == 0) {
+    {
+      const uint32_t on = lane == 0;
       const uint32_t id_g = make_idesc_f16(1, 0, 0, SD_Q, SD_Q);
       const uint32_t id_y = make_idesc_f16(1, 0, 1, SD_Q, PP);
       const uint32_t id_y2 = make_idesc_f16(1, 0, 1, SD_Q, PP * K::NY2);
@@ -162,13 +198,13 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       const uint64_t d_s = make_smem_desc_sw128(smem_u32(sShi), SD_N * 128, 1024), d_xw = make_smem_desc_sw128(smem_u32(sXhi), SD_Q * 128, 1024);
       auto scores = [&](int c) {
         const uint64_t dc = d_st + (c % K::STAGES) * (K::STAGE >> 4);
-        const uint32_t to = tm + (c % K::NG) * 128;
+        const uint32_t to = (c % K::NG) * 128;
 #pragma unroll
         for (int kk = 0; kk < SD_N / 16; ++kk) {
           const uint32_t off = (kk >> 2) * 1024 + (kk & 3) * 2;
-          umma_f16(to, dc + off, dc + (K::TBC >> 4) + off, id_g, kk ? 1u : 0u);
+          sd_mma(on, to, dc + off, dc + (K::TBC >> 4) + off, id_g, kk ? 1u : 0u);
         }
-        umma_commit(g_full);
+        sd_commit(on, g_full);
       };
       bool ok = true;
       if (!so) {
@@ -187,7 +223,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
           for (int part = 0; part < 2 / K::NY2; ++part)
 #pragma unroll
             for (int kk = 0; kk < SD_N / 16; ++kk)
-              umma_f16(tm + K::COL_Y2, dc + (kk >> 2) * 1024 + (kk & 3) * 2, d_s + part * (K::TS >> 4) + kk * 128, id_y2, (part || kk) ? 1u : 0u);
+              sd_mma(on, K::COL_Y2, dc + (kk >> 2) * 1024 + (kk & 3) * 2, d_s + part * (K::TS >> 4) + kk * 128, id_y2, (part || kk) ? 1u : 0u);
         }
         SD_WAIT(xw_ready, c & 1, ST_TIMEOUT_EMPTY);
         tc_fence_after();
@@ -195,21 +231,21 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
         for (int part = 0; part < 2; ++part)
 #pragma unroll
           for (int kk = 0; kk < SD_Q / 16; ++kk)
-            umma_f16(tm + K::COL_S, dmn + (K::TBC >> 4) + kk * 128, d_xw + part * (K::TX >> 4) + kk * 128, id_s, 1u);
-        umma_commit(s_full);
+            sd_mma(on, K::COL_S, dmn + (K::TBC >> 4) + kk * 128, d_xw + part * (K::TX >> 4) + kk * 128, id_s, 1u);
+        sd_commit(on, s_full);
         if (!so) {
           SD_WAIT(m_ready, c & 1, ST_TIMEOUT_TMEM_EMPTY);
           tc_fence_after();
-          const uint32_t m0 = tm + (c % K::NG) * 128;
+          const uint32_t m0 = (c % K::NG) * 128;
 #pragma unroll
           for (int part = 0; part < 2; ++part)
 #pragma unroll
             for (int kk = 0; kk < SD_Q / 16; ++kk)
-              umma_f16_ts(tm + K::COL_Y, m0 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8, dmn + (2 * K::TBC >> 4) + kk * 128, id_y,
+              sd_mma_ts(on, K::COL_Y, m0 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8, dmn + (2 * K::TBC >> 4) + kk * 128, id_y,
                           (part || kk) ? 1u : 0u);
-          umma_commit(y_full);
+          sd_commit(on, y_full);
         }
-        umma_commit(&empty[s]);
+        sd_commit(on, &empty[s]);
         if (!so && c + 1 < nc) {
           if (K::NG == 1) SD_WAIT(y_full, c & 1, ST_TIMEOUT_TMEM_FULL);      // the one score buffer still holds this chunk's weights
           SD_WAIT(&full[(c + 1) % K::STAGES], ((c + 1) / K::STAGES) & 1, ST_TIMEOUT_FULL);
@@ -475,7 +511,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
     for (int k = 0; k < 64; ++k) __nanosleep(1000);
     __syncthreads();
   }
-  if (warp == SD_W_MMA) { tc_fence_after(); tmem_dealloc(tm, 512); }
+  if (warp == SD_W_MMA) { tc_fence_after(); tmem_dealloc(*tmem_slot, 512); }
 }
 
 // ws slots 1 .. n_seg - 1 from "what segment k adds" to "state before the segment"; one thread per state value.

@@ -29,7 +29,7 @@ SIZES = {   # width, ff, query heads, kv heads, head size, mamba heads, groups, 
     "m": dict(width=2560, ff=6912, H=20, G=5, hd=128, mh=80, mg=1, layers=12),
     "l": dict(width=4096, ff=14336, H=32, G=8, hd=128, mh=128, mg=8, layers=8),
 }
-WINDOW, KEEP, VOCAB, STATE, VDIM = 1024, 4, 32000, 128, 64
+WINDOW, KEEP, VOCAB, STATE, VDIM = 1024, 8, 32000, 128, 64
 
 
 def peaks():
@@ -51,7 +51,7 @@ def layer_config(z, layers=None):
                                                   "norm_groups": z["mg"]}}
     n = layers or z["layers"]
     return LayerListConfig.from_json({"architecture": "Zikedra", "layers": [at if i % 4 == 3 else mb for i in range(n)], "width": z["width"],
-                                      "vocab": VOCAB, "norm": {"eps": 1e-5}, "logit_softcap": 15.0})
+                                      "vocab": VOCAB, "norm": {"eps": 1e-5}, "logit_softcap": 30.0})
 
 
 def dense_config(z, layers=None):
@@ -217,7 +217,7 @@ def token_kernels(t, z, m, mem, T):
     gemv("GEMV: output (gated norm inside)", "GEMV", w0.w_o, True, prologue=3, d=n, v32=gv, sq=sq, n_sq=2 * ma.H, w1=w0.vec["norm"], parts=z["mg"])
     gemv("GEMV: gate/up + SwiGLU", "GEMV: gate/up + SwiGLU", w0.w_gu, swiglu=1, **res)
     gemv("GEMV: down", "GEMV", w0.w_down, True, prologue=0, d=E, x16=aa, ldx=E)
-    gemv("GEMV: vocabulary (both norms inside)", "GEMV: vocabulary", m.head, True, w2=m.final_norm, softcap=15.0, **res)
+    gemv("GEMV: vocabulary (both norms inside)", "GEMV: vocabulary", m.head, True, w2=m.final_norm, softcap=30.0, **res)
     cb = 2 * WINDOW * Gq * hd * 2
     kv = [(mem.layers[3].k.clone(), mem.layers[3].v.clone()) for _ in range(16)]
 

@@ -4,7 +4,7 @@
 
 Standard input holds one JSON object a line,
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 0, "entries": [{"id": "a", "tokens": [811, 40, 9, 40], "want": [1, 3]}], "end": []}
 
 ``entries``: for each request its next tokens and the places among them whose logits are wanted; ``end``: requests that
 are finished after the step.  Logits go to ``<out>/<step>.f32`` (little-endian fp32, [wanted, vocab], in the order of the

@@ -1,4 +1,4 @@
-// Attention of layer-list models on CUDA cores (contract in gb_layers.h): what every head size and fp32 run on, and the
+// Attention of layer-list models on CUDA cores (interface in gb_layers.h): what every head size and fp32 run on, and the
 // token step.  Keys live in one cache per layer: the first `keep` positions stay, later positions share a ring.  The keys
 // a query range can see are enumerated as one list (kept positions, then the window), so no slot outside it is read.
 #include <type_traits>

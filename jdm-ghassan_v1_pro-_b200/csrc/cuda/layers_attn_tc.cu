@@ -1,4 +1,4 @@
-// Prompt attention of layer-list models on the tensor cores (contract in gb_layers.h): queries of the new tokens against
+// Prompt attention of layer-list models on the tensor cores (interface in gb_layers.h): queries of the new tokens against
 // the layer's cache (kept first positions + ring), bf16 operands, fp32 scores, weights and sums.
 //
 // Work split as in attention_tc.cu: warp 4 = TMA producer, warp 5 = MMA issuer, warps 0-3 = one soft-max thread per query

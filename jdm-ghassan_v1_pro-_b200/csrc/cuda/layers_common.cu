@@ -1,4 +1,4 @@
-// Row-wise kernels of layer-list models (contract in gb_layers.h): embedding, norms on sublayer outputs with the residual
+// Row-wise kernels of layer-list models (interface in gb_layers.h): embedding, norms on sublayer outputs with the residual
 // add, the fp32 matrix product, the fp32 SwiGLU, the logit cap.
 #include <type_traits>
 

@@ -1,4 +1,4 @@
-// Token-step matrix-vector products of layer-list models (contract in gb_layers.h).  One token is bound by weight bytes
+// Token-step matrix-vector products of layer-list models (interface in gb_layers.h).  One token is bound by weight bytes
 // and by the number of dependent launches, so what lies between two products (residual add with the norm of the
 // sublayer's output, gated group norm, final norm) is the prologue of the second one: every block makes the input
 // vector it needs in shared memory, and one block writes the new residual for the kernels after it.  Weights do not depend

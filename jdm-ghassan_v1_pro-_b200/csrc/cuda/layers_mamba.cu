@@ -1,4 +1,4 @@
-// Mamba-2 mixer of layer-list models (contract in gb_layers.h): causal convolution with its carried inputs, the state
+// Mamba-2 mixer of layer-list models (interface in gb_layers.h): causal convolution with its carried inputs, the state
 // recurrence token by token (fp32 for every size; the chunked tensor-core form is in layers_ssd.cu), the gated group
 // norm, and the one-token step that fuses convolution and recurrence.
 //

@@ -1,4 +1,4 @@
-// Mamba-2 state recurrence over many tokens on the tensor cores (contract in gb_layers.h): chunks of 128 tokens, the
+// Mamba-2 state recurrence over many tokens on the tensor cores (interface in gb_layers.h): chunks of 128 tokens, the
 // state of a head resident in tensor memory from chunk to chunk.
 //
 // With L_t the running sum of the log decays inside a chunk (fp32), the chunk's outputs and its new state are

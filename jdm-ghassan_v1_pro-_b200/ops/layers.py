@@ -1,4 +1,4 @@
-"""Launchers for the kernels of layer-list models (``csrc/cuda/layers_*.cu``; contract in ``gb_layers.h``)."""
+"""Launchers for the kernels of layer-list models (``csrc/cuda/layers_*.cu``; interface in ``gb_layers.h``)."""
 from __future__ import annotations
 
 import ctypes

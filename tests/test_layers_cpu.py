@@ -207,12 +207,12 @@ def test_trace_protocol(tmp_path):
         def end(self, key):
             self.log.append(("end", key))
 
-    lines = [json.dumps({"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}), "",
+    lines = [json.dumps({"step": 0, "entries": [{"id": "a", "tokens": [8, 40, 9, 41], "want": [1, 3]}], "end": []}), "",
              json.dumps({"step": 1, "entries": [{"id": "a", "tokens": [4], "want": []}], "end": ["a"]})]
     eng, said = Fake(), []
     trace.run(eng, lines, str(tmp_path), said.append)
-    assert said == ["done 0", "done 1"] and eng.log == [("step", "a", [5, 17, 3]), ("step", "a", [4]), ("end", "a")]
-    assert np.fromfile(tmp_path / "0.f32", "<f4").tolist() == [5.0, 0.5, 3.0, 0.5] and not (tmp_path / "1.f32").exists()
+    assert said == ["done 0", "done 1"] and eng.log == [("step", "a", [8, 40, 9, 41]), ("step", "a", [4]), ("end", "a")]
+    assert np.fromfile(tmp_path / "0.f32", "<f4").tolist() == [40.0, 0.5, 41.0, 0.5] and not (tmp_path / "1.f32").exists()
     with pytest.raises(SystemExit):
         trace._parser().parse_args(["--model", "m", "--out", "o", "--dtype", "int8"])
 

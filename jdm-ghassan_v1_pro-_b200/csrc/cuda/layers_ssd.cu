@@ -82,6 +82,32 @@ __device__ __forceinline__ void sd_commit(uint32_t on, uint64_t* bar) {
       : "memory");
 }
 
+// Out of line: the kernel has five roles with long straight-line bodies, and what bounds it once the chains overlap is the
+// instruction cache (a wait that was over cost 400 cycles with everything unrolled and inlined).
+__device__ __noinline__ bool sd_wait(uint32_t bar, uint32_t parity, int* status, int code, volatile int* abort_flag) {
+  const long long t0 = clock64();
+  for (;;) {
+#pragma unroll 1
+    for (int i = 0; i < 1024; ++i) {
+      uint32_t ok;
+      asm volatile(
+          "{\n\t.reg .pred P1;\n\t"
+          "mbarrier.try_wait.parity.shared::cta.b64 P1, [%1], %2;\n\t"
+          "selp.b32 %0, 1, 0, P1;\n\t}"
+          : "=r"(ok)
+          : "r"(bar), "r"(parity)
+          : "memory");
+      if (ok) return true;
+    }
+    if (*abort_flag) return false;
+    if (clock64() - t0 > 4000000000LL) {
+      atomicCAS(status, 0, code);
+      *abort_flag = 1;
+      return false;
+    }
+  }
+}
+
 // 2 values -> packed bf16 pair and the packed remainders
 __device__ __forceinline__ void sd_split2(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = Cvt<__nv_bfloat16>::pack2(a, b);
@@ -167,7 +193,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
   constexpr uint32_t tm = 0;
   if (*tmem_slot != 0 && threadIdx.x == 0) { atomicCAS(p.status, 0, ST_BAD_ARGUMENT); *abort_flag = 1; }
   const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
-#define SD_WAIT(bar, ph, code) if (!at_wait(bar, ph, p.status, code, abort_flag)) break
+#define SD_WAIT(bar, ph, code) if (!sd_wait(smem_u32(bar), ph, p.status, code, abort_flag)) break
 
   if (warp == SD_W_TMA) {
     // ------------------------------------------------------------------ TMA
@@ -208,7 +234,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       };
       bool ok = true;
       if (!so) {
-        ok = at_wait(&full[0], 0, p.status, ST_TIMEOUT_FULL, abort_flag);
+        ok = sd_wait(smem_u32(&full[0]), 0, p.status, ST_TIMEOUT_FULL, abort_flag);
         if (ok) { tc_fence_after(); scores(0); }
       }
       for (int c = 0; c < nc && ok; ++c) {
@@ -303,9 +329,8 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       // weights (C_t . B_s) exp(L_t - L_s) dt_s, written over the scores they come from: per 32 columns, 16 columns of
       // packed values and 16 of packed remainders.  Left of the diagonal block the exponential is a product of a factor
       // of the row and one of the column, both against the L at the end of the column's block (neither exceeds 1).
-#pragma unroll
-      for (int q0 = 0; q0 < 4; q0 += 2) {
-        const int q = q0 + half;
+#pragma unroll 1
+      for (int q = half; q < 4; q += 2) {
         uint32_t hi[16], lo[16];
         if (q < quarter) {
           uint32_t rg[32];
@@ -353,23 +378,22 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       SD_WAIT(y_full, c & 1, ST_TIMEOUT_TMEM_FULL);
       SD_WAIT(&full[s], (c / K::STAGES) & 1, ST_TIMEOUT_FULL);      // long since true; this thread reads x itself
       tc_fence_after();
-#pragma unroll
-      for (int q0 = 0; q0 < PP / 64; ++q0) {
-        const int c0 = half * (PP / 2) + q0 * 32;
-        uint32_t a[32], e[32];
-        tmem_ld_32x32(tm + K::COL_Y + lane_base + c0, a);
-        tmem_ld_32x32(tm + K::COL_Y2 + lane_base + c0, e);
+#pragma unroll 1
+      for (int c0 = half * (PP / 2); c0 < (half + 1) * (PP / 2); c0 += 16) {
+        uint32_t a[16], e[16];
+        tmem_ld_32x16(tm + K::COL_Y + lane_base + c0, a);
+        tmem_ld_32x16(tm + K::COL_Y2 + lane_base + c0, e);
         if constexpr (K::NY2 == 2) {
-          uint32_t e2[32];
-          tmem_ld_32x32(tm + K::COL_Y2 + PP + lane_base + c0, e2);
+          uint32_t e2[16];
+          tmem_ld_32x16(tm + K::COL_Y2 + PP + lane_base + c0, e2);
           tmem_ld_wait();
 #pragma unroll
-          for (int k = 0; k < 32; ++k) e[k] = __float_as_uint(__uint_as_float(e[k]) + __uint_as_float(e2[k]));
+          for (int k = 0; k < 16; ++k) e[k] = __float_as_uint(__uint_as_float(e[k]) + __uint_as_float(e2[k]));
         } else {
           tmem_ld_wait();
         }
 #pragma unroll
-        for (int k = 0; k < 4 && live; ++k) {
+        for (int k = 0; k < 2 && live; ++k) {
           const int col = c0 + 8 * k;
           const uint4 xq = *reinterpret_cast<const uint4*>(sx + (col >> 6) * (SD_Q * 128) + sw128_off(r, col & 63));
           const uint32_t xw[4] = {xq.x, xq.y, xq.z, xq.w};
@@ -432,7 +456,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       total += Ll;
       if (c > 0) SD_WAIT(s_full, (c - 1) & 1, ST_TIMEOUT_TMEM_FULL);
       tc_fence_after();
-#pragma unroll
+#pragma unroll 1
       for (int q = 0; q < PP / 32; ++q) {
         uint32_t v[32];
         tmem_ld_32x32(ts + q * 32, v);
@@ -467,7 +491,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       if (lane == 0) mbar_arrive(s_ready);
       SD_WAIT(&full[s], (c / K::STAGES) & 1, ST_TIMEOUT_FULL);
       const uint8_t* sx = smem + s * K::STAGE + 2 * K::TBC;
-#pragma unroll
+#pragma unroll 4
       for (int q = 0; q < PP / 8; ++q) {
         const uint32_t off = (q >> 3) * (SD_Q * 128) + sw128_off(r, (q & 7) * 8);
         const uint4 xq = *reinterpret_cast<const uint4*>(sx + off);
@@ -486,7 +510,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       if (lane == 0) { mbar_arrive(xw_ready); mbar_arrive(&l_empty[ls]); }
       ok = true;
     }
-    if (ok && nc > 0 && at_wait(s_full, (nc - 1) & 1, p.status, ST_TIMEOUT_TMEM_FULL, abort_flag)) {
+    if (ok && nc > 0 && sd_wait(smem_u32(s_full), (nc - 1) & 1, p.status, ST_TIMEOUT_TMEM_FULL, abort_flag)) {
       tc_fence_after();
       float* dst = so ? ws + (seg + 1) * per : (seg == p.n_seg - 1 ? home : nullptr);
 #pragma unroll 1

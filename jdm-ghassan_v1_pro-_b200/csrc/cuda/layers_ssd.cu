@@ -26,8 +26,6 @@ namespace gb {
 
 constexpr int SD_Q = 128;                  // tokens per chunk
 constexpr int SD_N = 128;                  // padded state size
-constexpr int SD_W_STATE = 8, SD_W_TMA = 12, SD_W_MMA = 13, SD_W_DT = 14;
-constexpr int SD_THREADS = 480;
 
 struct SsdParams {
   int B, n, H, P, N, G, Ns;
@@ -36,7 +34,7 @@ struct SsdParams {
   float* ssm;
   __nv_bfloat16* y; long long ld_y;
   const gb_seq_state* st;
-  int n_chunks, seg_chunks, n_seg, state_only;
+  int n_chunks, seg_chunks, n_seg;
   float* ws_state;                         // [B, H, n_seg, P, Ns]: slot k = state before segment k (first launch: slot 0 as it
                                            // is, slot k + 1 = what segment k adds from zero)
   float* ws_decay;                         // [B, H, n_seg]: log2 decay over segment k
@@ -115,26 +113,31 @@ __device__ __forceinline__ void sd_split2(float a, float b, uint32_t& hi, uint32
   lo = Cvt<__nv_bfloat16>::pack2(a - h.x, b - h.y);
 }
 
-template <int PP>
+// SO: the state-only pass, without the token-row warps, C, and the state as an operand: two CTAs share an SM (head size 64).
+template <int PP, bool SO>
 struct SsdCfg {
-  static constexpr int STAGES = PP == 64 ? 2 : 1;
+  static constexpr int W_STATE = SO ? 0 : 8, W_TMA = W_STATE + 4, W_MMA = W_STATE + 5, W_DT = W_STATE + 6;
+  static constexpr int THREADS = (W_DT + 1) * 32, CTAS = SO && PP == 64 ? 2 : 1;
+  static constexpr int STAGES = !SO && PP == 64 ? 2 : 1;
   static constexpr int NG = PP == 64 ? 2 : 1;                       // score buffers in tensor memory
-  static constexpr uint32_t TBC = SD_Q * SD_N * 2, TX = SD_Q * PP * 2, STAGE = 2 * TBC + TX;
-  static constexpr uint32_t TS = SD_N * PP * 2;
+  static constexpr uint32_t TBC = SD_Q * SD_N * 2, TX = SD_Q * PP * 2;
+  static constexpr uint32_t OFF_B = SO ? 0 : TBC, OFF_X = OFF_B + TBC, STAGE = OFF_X + TX;      // a stage: C, B, x
+  static constexpr uint32_t TS = SO ? 0 : SD_N * PP * 2;
   static constexpr size_t TILES = (size_t)STAGES * STAGE + 2 * TS + 2 * TX;
   static constexpr size_t SMEM = TILES + 2 * (2 * SD_Q + 96) * 4 + 128;
   // the products with both terms of S_prev side by side (one pass over C) where tensor memory has the columns
   static constexpr int NY2 = PP == 64 ? 2 : 1;
-  static constexpr int COL_Y = 128 * NG, COL_Y2 = COL_Y + PP, COL_S = COL_Y2 + PP * NY2;
+  static constexpr int COL_Y = 128 * NG, COL_Y2 = COL_Y + PP, COL_S = SO ? 0 : COL_Y2 + PP * NY2;
+  static constexpr int COLS = SO ? PP : 512;
 };
 
-template <int PP>
-__global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_constant__ CUtensorMap tmX,
+template <int PP, bool SO>
+__global__ void __launch_bounds__(SsdCfg<PP, SO>::THREADS, SsdCfg<PP, SO>::CTAS) ll_ssd_kernel(const __grid_constant__ CUtensorMap tmX,
                                                                const __grid_constant__ CUtensorMap tmB,
                                                                const __grid_constant__ CUtensorMap tmC,
                                                                const __grid_constant__ SsdParams p) {
   using T = __nv_bfloat16;
-  using K = SsdCfg<PP>;
+  using K = SsdCfg<PP, SO>;
   extern __shared__ __align__(1024) uint8_t smem[];
   if (smem_u32(smem) & 1023u) {            // no static shared memory: the dynamic window starts aligned
     if (threadIdx.x == 0) atomicCAS(p.status, 0, ST_BAD_ARGUMENT);
@@ -163,7 +166,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const bool so = p.state_only != 0;
+  constexpr bool so = SO;
   const int seg = blockIdx.x % (so ? p.n_seg - 1 : p.n_seg), bh = blockIdx.x / (so ? p.n_seg - 1 : p.n_seg);
   const int b = bh / p.H, h = bh - b * p.H, g = h / (p.H / p.G);
   const int c_lo = seg * p.seg_chunks, c_hi = min(p.n_chunks, c_lo + p.seg_chunks), nc = c_hi - c_lo;
@@ -185,17 +188,17 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
     *abort_flag = 0;
     fence_barrier_init();
   }
-  if (warp == SD_W_MMA) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
+  if (warp == K::W_MMA) { tmem_alloc(tmem_slot, K::COLS); tmem_relinquish(); }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  // all 512 columns are this CTA's, so the allocation starts at column 0 (checked: addresses below are constants)
-  constexpr uint32_t tm = 0;
-  if (*tmem_slot != 0 && threadIdx.x == 0) { atomicCAS(p.status, 0, ST_BAD_ARGUMENT); *abort_flag = 1; }
+  // with all 512 columns the allocation starts at column 0 (checked), and the addresses below are constants
+  const uint32_t tm = so ? *tmem_slot : 0u;
+  if (!so && *tmem_slot != 0 && threadIdx.x == 0) { atomicCAS(p.status, 0, ST_BAD_ARGUMENT); *abort_flag = 1; }
   const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
 #define SD_WAIT(bar, ph, code) if (!sd_wait(smem_u32(bar), ph, p.status, code, abort_flag)) break
 
-  if (warp == SD_W_TMA) {
+  if (warp == K::W_TMA) {
     // ------------------------------------------------------------------ TMA
     if (lane == 0) {
       for (int c = 0; c < nc; ++c) {
@@ -203,14 +206,14 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
         SD_WAIT(&empty[s], ph ^ 1, ST_TIMEOUT_EMPTY);
         uint8_t* st = smem + s * K::STAGE;
         const int row = b * p.n + (c_lo + c) * SD_Q;
-        mbar_arrive_expect_tx(&full[s], so ? K::TBC + K::TX : K::STAGE);
-        load_tile<SD_N>(&tmB, &full[s], st + K::TBC, g * SD_N, row);
-        load_tile<PP>(&tmX, &full[s], st + 2 * K::TBC, h * PP, row);
+        mbar_arrive_expect_tx(&full[s], K::STAGE);
+        load_tile<SD_N>(&tmB, &full[s], st + K::OFF_B, g * SD_N, row);
+        load_tile<PP>(&tmX, &full[s], st + K::OFF_X, h * PP, row);
         if (!so) load_tile<SD_N>(&tmC, &full[s], st, g * SD_N, row);
       }
     }
     __syncwarp();
-  } else if (warp == SD_W_MMA) {
+  } else if (warp == K::W_MMA) {
     // ------------------------------------------------------------------ MMA
     {
       const uint32_t on = lane == 0;
@@ -228,7 +231,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
 #pragma unroll
         for (int kk = 0; kk < SD_N / 16; ++kk) {
           const uint32_t off = (kk >> 2) * 1024 + (kk & 3) * 2;
-          sd_mma(on, to, dc + off, dc + (K::TBC >> 4) + off, id_g, kk ? 1u : 0u);
+          sd_mma(on, to, dc + off, dc + (K::OFF_B >> 4) + off, id_g, kk ? 1u : 0u);
         }
         sd_commit(on, g_full);
       };
@@ -257,7 +260,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
         for (int part = 0; part < 2; ++part)
 #pragma unroll
           for (int kk = 0; kk < SD_Q / 16; ++kk)
-            sd_mma(on, K::COL_S, dmn + (K::TBC >> 4) + kk * 128, d_xw + part * (K::TX >> 4) + kk * 128, id_s, 1u);
+            sd_mma(on, tm + K::COL_S, dmn + (K::OFF_B >> 4) + kk * 128, d_xw + part * (K::TX >> 4) + kk * 128, id_s, 1u);
         sd_commit(on, s_full);
         if (!so) {
           SD_WAIT(m_ready, c & 1, ST_TIMEOUT_TMEM_EMPTY);
@@ -267,7 +270,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
           for (int part = 0; part < 2; ++part)
 #pragma unroll
             for (int kk = 0; kk < SD_Q / 16; ++kk)
-              sd_mma_ts(on, K::COL_Y, m0 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8, dmn + (2 * K::TBC >> 4) + kk * 128, id_y,
+              sd_mma_ts(on, K::COL_Y, m0 + (kk >> 1) * 32 + part * 16 + (kk & 1) * 8, dmn + (K::OFF_X >> 4) + kk * 128, id_y,
                           (part || kk) ? 1u : 0u);
           sd_commit(on, y_full);
         }
@@ -281,7 +284,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       }
     }
     __syncwarp();
-  } else if (warp == SD_W_DT) {
+  } else if (warp == K::W_DT) {
     // ------------------------------------------------------------------ dt and L
     const float bias = p.dt_bias[h], na2 = -expf(p.A_log[h]) * 1.4426950408889634f;
     for (int c = 0; c < nc; ++c) {
@@ -314,7 +317,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       if (lane == 0) mbar_arrive(&l_full[s]);
     }
     __syncwarp();
-  } else if (warp < SD_W_STATE) {
+  } else if (warp < K::W_STATE) {
     // ------------------------------------------------------------------ token rows
     const int quarter = warp & 3, half = warp >> 2, r = quarter * 32 + lane;
     const float D = p.D[h];
@@ -371,7 +374,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(m_ready);
       const float eL = sd_ex2(L);
-      const uint8_t* sx = smem + s * K::STAGE + 2 * K::TBC;
+      const uint8_t* sx = smem + s * K::STAGE + K::OFF_X;
       T* yp = p.y + ((long long)b * p.n + t) * p.ld_y + h * p.P;
       const bool live = t < p.n;
       const bool vec = p.P == PP && ((reinterpret_cast<uintptr_t>(p.y) | (uintptr_t)(p.ld_y * 2)) & 15) == 0;
@@ -423,7 +426,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
     }
   } else {
     // ------------------------------------------------------------------ state rows and scaled x
-    const int r = threadIdx.x - SD_W_STATE * 32;   // state column (0 .. 127) / token of the chunk
+    const int r = threadIdx.x - K::W_STATE * 32;   // state column (0 .. 127) / token of the chunk
     const bool live_n = r < p.N;
     const long long per = (long long)p.P * p.Ns;
     float* home = p.ssm + bh * per;
@@ -490,7 +493,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(s_ready);
       SD_WAIT(&full[s], (c / K::STAGES) & 1, ST_TIMEOUT_FULL);
-      const uint8_t* sx = smem + s * K::STAGE + 2 * K::TBC;
+      const uint8_t* sx = smem + s * K::STAGE + K::OFF_X;
 #pragma unroll 4
       for (int q = 0; q < PP / 8; ++q) {
         const uint32_t off = (q >> 3) * (SD_Q * 128) + sw128_off(r, (q & 7) * 8);
@@ -535,7 +538,7 @@ __global__ void __launch_bounds__(SD_THREADS, 1) ll_ssd_kernel(const __grid_cons
     for (int k = 0; k < 64; ++k) __nanosleep(1000);
     __syncthreads();
   }
-  if (warp == SD_W_MMA) { tc_fence_after(); tmem_dealloc(*tmem_slot, 512); }
+  if (warp == K::W_MMA) { tc_fence_after(); tmem_dealloc(*tmem_slot, K::COLS); }
 }
 
 // ws slots 1 .. n_seg - 1 from "what segment k adds" to "state before the segment"; one thread per state value.
@@ -555,14 +558,14 @@ __global__ void __launch_bounds__(256) ll_ssd_combine_kernel(float* __restrict__
 struct SsdPlan { int n_chunks, seg_chunks, n_seg; };
 
 // Segments per head: the cheapest number of rounds over the SMs.  A CTA costs about three chunks to start and drain; a
-// state-only chunk about 0.7 of a full one.
+// state-only chunk about 0.7 of a full one, and two state-only CTAs share an SM.
 static SsdPlan ssd_plan(int BH, int n, int sms) {
   SsdPlan best{(n + SD_Q - 1) / SD_Q, 0, 1};
   best.seg_chunks = best.n_chunks;
   double cost = (double)((BH + sms - 1) / sms) * (best.n_chunks + 3.0);
   for (int s = 2; s <= 16 && s <= best.n_chunks; ++s) {
     const int per = (best.n_chunks + s - 1) / s, k = (best.n_chunks + per - 1) / per;
-    const double c = (per + 3.0) * ((BH * k + sms - 1) / sms) + (0.7 * per + 3.0) * ((BH * (k - 1) + sms - 1) / sms) + 3.0;
+    const double c = (per + 3.0) * ((BH * k + sms - 1) / sms) + (0.7 * per + 3.0) * ((BH * (k - 1) + 2 * sms - 1) / (2 * sms)) + 3.0;
     if (c < cost * 0.95) { cost = c; best.seg_chunks = per; best.n_seg = k; }
   }
   return best;
@@ -577,17 +580,24 @@ static int ssd_sms() {
   return sms;
 }
 
+template <int PP, bool SO>
+static int ssd_attr() {
+  static bool done = false;
+  if (!done) {
+    if (cudaFuncSetAttribute(ll_ssd_kernel<PP, SO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SsdCfg<PP, SO>::SMEM) != cudaSuccess) return -10;
+    if (SO) (void)cudaFuncSetAttribute(ll_ssd_kernel<PP, SO>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+    done = true;
+  }
+  return 0;
+}
+
 template <int PP>
 static int ssd_go(const gb_ll_mamba_args& a, int force_segments, cudaStream_t st) {
-  using K = SsdCfg<PP>;
-  static_assert(K::SMEM <= 232448 && K::COL_S + PP <= 512, "shared memory / tensor memory budget");
+  using K = SsdCfg<PP, false>;
+  using KS = SsdCfg<PP, true>;
+  static_assert(K::SMEM <= 232448 && K::COL_S + PP <= 512 && KS::CTAS * (KS::SMEM + 1024) <= 233472, "shared memory / tensor memory budget");
   const int sms = ssd_sms();
-  if (sms <= 0) return -10;
-  static bool attr = false;
-  if (!attr) {
-    if (cudaFuncSetAttribute(ll_ssd_kernel<PP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)K::SMEM) != cudaSuccess) return -10;
-    attr = true;
-  }
+  if (sms <= 0 || ssd_attr<PP, false>() || ssd_attr<PP, true>()) return -10;
   CUtensorMap tx, tb, tc;
   const uint64_t rows = (uint64_t)a.B * a.n;
   if (gb_make_tmap_2d_16b(&tx, a.xh, rows, (uint64_t)a.H * PP, (uint64_t)a.H * PP, SD_Q, 64, 1)) return -20;
@@ -610,13 +620,11 @@ static int ssd_go(const gb_ll_mamba_args& a, int force_segments, cudaStream_t st
   if (plan.n_seg > 1) {
     p.ws_state = a.chunk_ws;
     p.ws_decay = a.chunk_ws + BH * plan.n_seg * a.P * a.Ns;
-    p.state_only = 1;
-    ll_ssd_kernel<PP><<<(unsigned)(BH * (plan.n_seg - 1)), SD_THREADS, K::SMEM, st>>>(tx, tb, tc, p);
-    p.state_only = 0;
+    ll_ssd_kernel<PP, true><<<(unsigned)(BH * (plan.n_seg - 1)), KS::THREADS, KS::SMEM, st>>>(tx, tb, tc, p);
     const long long per = (long long)a.P * a.Ns;
     ll_ssd_combine_kernel<<<dim3((unsigned)((per + 255) / 256), (unsigned)BH), 256, 0, st>>>(p.ws_state, p.ws_decay, plan.n_seg, per);
   }
-  ll_ssd_kernel<PP><<<(unsigned)(BH * plan.n_seg), SD_THREADS, K::SMEM, st>>>(tx, tb, tc, p);
+  ll_ssd_kernel<PP, false><<<(unsigned)(BH * plan.n_seg), K::THREADS, K::SMEM, st>>>(tx, tb, tc, p);
   return gb_launch_rc();
 }
 

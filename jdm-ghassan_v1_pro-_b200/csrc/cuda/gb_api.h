@@ -23,7 +23,8 @@ typedef struct gb_gemm_args {
   int b_mn_major;           // 0: stored [N,K]; 1: stored [K,N]
   int is_bf16;              // operand type: 0 fp16, 1 bf16
   int out_dtype;            // 0 fp16, 1 bf16, 2 fp32
-  int epilogue;             // 0 store (+ optional fp32 addend), 1 SwiGLU forward, 2 SwiGLU backward
+  int epilogue;             // 0 store (+ optional fp32 addend), 1 SwiGLU forward, 2 SwiGLU backward, 4 store of the
+                            // squared positive part (mode 0, bf16)
   int block_n;              // 64 / 128 / 256 (0 = 128)
   int mode;                 // 0 dense, 1 grouped over rows (tile map), 2 grouped over the reduction dim
   const int* tile_expert;   // mode 1

@@ -31,7 +31,7 @@ static constexpr uint32_t SLOT_BYTES = 4096;   // 32 rows x 128 bytes
 static constexpr uint32_t TMEM_COLS = 512;
 static constexpr uint32_t BAR_BYTES = 512;
 
-enum { EPI_STORE = 0, EPI_SWIGLU_FWD = 1, EPI_SWIGLU_BWD = 2 };
+enum { EPI_STORE = 0, EPI_SWIGLU_FWD = 1, EPI_SWIGLU_BWD = 2, EPI_RELU2 = 4 };   // numbered as in gemm_sm100.cu
 
 struct Params {
   int M, N, K;
@@ -133,7 +133,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   }
   if (warp == W_TMA && lane == 0) {
     tma_prefetch_desc(&tmA); tma_prefetch_desc(&tmB); tma_prefetch_desc(&tmO);
-    if (EPI != EPI_STORE) tma_prefetch_desc(&tmX);
+    if (EPI != EPI_STORE && EPI != EPI_RELU2) tma_prefetch_desc(&tmX);
   }
   tc_fence_before();
   __syncthreads();
@@ -271,7 +271,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       }
       const uint32_t taddr = tmem_base + ab * TN + half * 128 + (uint32_t(quarter * 32) << 16);
 
-      if constexpr (EPI == EPI_STORE && sizeof(OutT) == 2) {
+      if constexpr ((EPI == EPI_STORE || EPI == EPI_RELU2) && sizeof(OutT) == 2) {
 #pragma unroll 1
         for (int c = 0; c < 2; ++c) {               // 64-column chunks
           uint32_t r0[32], r1[32];
@@ -282,6 +282,14 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           } else {
 #pragma unroll
             for (int i = 0; i < 32; ++i) { r0[i] = 0; r1[i] = 0; }
+          }
+          if constexpr (EPI == EPI_RELU2) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const float a = fmaxf(__uint_as_float(r0[i]), 0.f), b = fmaxf(__uint_as_float(r1[i]), 0.f);
+              r0[i] = __float_as_uint(a * a);
+              r1[i] = __float_as_uint(b * b);
+            }
           }
           uint8_t* slot = acquire();
 #pragma unroll
@@ -614,6 +622,13 @@ extern "C" int gb_gemm_pair(const gb_gemm_args* a, cudaStream_t st) {
       if (ot == 2) return launch_pair<pr::EPI_STORE, 5, 2, float>(ta, tb, to, tx, p, max_tiles, st);
       if (ot == 1) return launch_pair<pr::EPI_STORE, 5, 2, __nv_bfloat16>(ta, tb, to, tx, p, max_tiles, st);
       return launch_pair<pr::EPI_STORE, 5, 2, __half>(ta, tb, to, tx, p, max_tiles, st);
+    }
+    case pr::EPI_RELU2: {
+      if (ot != 1 || a->addend || a->mode != 0) return -25;
+      rc = gb_make_tmap_3d_box128(&to, a->out, ot, a->N, a->M, 1, a->ldo, 0, 32);
+      if (rc) return rc - 300;
+      tx = to;
+      return launch_pair<pr::EPI_RELU2, 5, 2, __nv_bfloat16>(ta, tb, to, tx, p, max_tiles, st);
     }
     case pr::EPI_SWIGLU_FWD: {
       if (a->N % 128 || ot == 2 || a->mode == 2) return -23;

@@ -40,7 +40,8 @@ struct GemmParams {
 };
 
 enum { EPI_STORE = 0, EPI_SWIGLU_FWD = 1, EPI_SWIGLU_BWD = 2,
-       EPI_STORE_TILED = 3 };   // EPI_STORE with per-tile destinations (16-bit output), chosen by the launcher
+       EPI_STORE_TILED = 3,     // EPI_STORE with per-tile destinations (16-bit output), chosen by the launcher
+       EPI_RELU2 = 4 };         // EPI_STORE of the squared positive part (16-bit output)
 
 __device__ __forceinline__ bool wait_or_flag(uint64_t* bar, uint32_t parity, int* status, int code, volatile int* abort_flag) {
   long long t0 = clock64();
@@ -284,7 +285,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       const int row = t.a_row0 + r_in_tile;
       const bool row_ok = row < p.M;
       const uint32_t taddr0 = tmem_base + ab * BN + (uint32_t(quarter * 32) << 16);
-      if constexpr (EPI == EPI_STORE || EPI == EPI_STORE_TILED) {
+      if constexpr (EPI == EPI_STORE || EPI == EPI_STORE_TILED || EPI == EPI_RELU2) {
         // per-tile destinations: the rows of this tile go to wherever the table says (expert-parallel combine
         // writes them straight into the buffer of the GPU that owns the tokens)
         OutT* orow = p.tile_out ? reinterpret_cast<OutT*>(p.tile_out[t.tm]) + (long long)r_in_tile * p.ldo
@@ -305,6 +306,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
             float v[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i) v[i] = empty_k ? 0.f : __uint_as_float(r[b][i]);
+            if constexpr (EPI == EPI_RELU2) {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) { v[i] = fmaxf(v[i], 0.f); v[i] *= v[i]; }
+            }
             const int col = t.n0 + (c0 + b) * 32;
             const int nvalid = p.N - col;
             if constexpr (EPI == EPI_STORE_TILED && sizeof(OutT) == 2) {
@@ -552,6 +557,9 @@ extern "C" int gb_gemm(const gb_gemm_args* a, cudaStream_t st) {
       if (ot == 1) return dispatch_bn<gb::EPI_SWIGLU_FWD, __nv_bfloat16, __nv_bfloat16>(bn == 256 ? 256 : 128, ta, tb, p, max_tiles, st);
       if (ot == 0) return dispatch_bn<gb::EPI_SWIGLU_FWD, __half, __half>(bn == 256 ? 256 : 128, ta, tb, p, max_tiles, st);
       return -1;
+    case gb::EPI_RELU2:
+      if (ot != 1 || a->addend || a->mode != 0) return -1;
+      return dispatch_bn<gb::EPI_RELU2, __nv_bfloat16, __nv_bfloat16>(bn, ta, tb, p, max_tiles, st);
     case gb::EPI_SWIGLU_BWD:
       if (ot == 1) return dispatch_bn<gb::EPI_SWIGLU_BWD, __nv_bfloat16, __nv_bfloat16>(bn, ta, tb, p, max_tiles, st);
       if (ot == 0) return dispatch_bn<gb::EPI_SWIGLU_BWD, __half, __half>(bn, ta, tb, p, max_tiles, st);

@@ -18,6 +18,17 @@ __device__ __forceinline__ float2 ll_rotation(int pos, double freq) {
   return make_float2(cs, sn);
 }
 
+__device__ __forceinline__ float ll_query_temperature(int pos, float coef, int every) {
+  return 1.f + coef * logf((float)((pos + 1) / every + 1));
+}
+
+// Score as the soft-max sees it: scaled, capped, less the slope times the distance.
+__device__ __forceinline__ float ll_score(float dot, float scale, float cap, float slope, int back) {
+  float s = dot * scale;
+  if (cap > 0.f) s = cap * tanhf(s / cap);
+  return s - slope * (float)back;
+}
+
 __global__ void __launch_bounds__(256) ll_rotations_kernel(const double* __restrict__ freq, int pairs, const gb_seq_state* __restrict__ st,
                                                            int n, long long total, float2* __restrict__ cs) {
   pdl_wait();
@@ -72,6 +83,11 @@ __global__ void __launch_bounds__(256) ll_qkv_store_vec_kernel(const __grid_cons
 #pragma unroll
     for (int e = 0; e < 8; ++e) v[e] *= inv;
   }
+  if (h < a.H && a.temp_every > 0) {
+    const float f = ll_query_temperature(pos, a.temp_coef, a.temp_every);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= f;
+  }
   if (live && c < dp) ll_store8(dst + c, v);
 }
 
@@ -122,6 +138,7 @@ __global__ void __launch_bounds__(256) ll_qkv_store_kernel(const __grid_constant
   }
   float inv = 1.f;
   if (a.qk_norm) inv = ll_inv_rms(warp_sum(ss), a.dk, a.eps);
+  if (h < a.H && a.temp_every > 0) inv *= ll_query_temperature(pos, a.temp_coef, a.temp_every);
 #pragma unroll
   for (int k = 0; k < 8; ++k) {
     const int i = lane + 32 * k;
@@ -168,6 +185,7 @@ __global__ void __launch_bounds__(128) ll_attn_prefill_kernel(const __grid_const
     o[d] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
+  const float slope = a.slopes ? a.slopes[h] : 0.f;
   const LlKeyRange kr = ll_key_range(p0 + q0, p0 + min(a.n, q0 + ROWS) - 1, a.window, a.keep);
   for (int e0 = 0; e0 < kr.count; e0 += KT) {
     __syncthreads();
@@ -178,11 +196,11 @@ __global__ void __launch_bounds__(128) ll_attn_prefill_kernel(const __grid_const
     __syncthreads();
     for (int x = threadIdx.x; x < KT * a.dkp; x += 128) {
       const int kk = x / a.dkp, c = x - kk * a.dkp, p = sPos[kk];
-      sK[x] = p < 0 ? 0.f : Cvt<T>::to_f(reinterpret_cast<const T*>(a.cache_k)[(((long long)b * a.cap + ll_ring_row(p, a.keep, a.cap)) * a.G + g) * a.dkp + c]);
+      sK[x] = p < 0 ? 0.f : Cvt<T>::to_f(reinterpret_cast<const T*>(a.cache_k)[((long long)b * a.cap + ll_ring_row(p, a.keep, a.cap)) * a.ld_k + g * a.dkp + c]);
     }
     for (int x = threadIdx.x; x < KT * a.dvp; x += 128) {
       const int kk = x / a.dvp, c = x - kk * a.dvp, p = sPos[kk];
-      sV[x] = p < 0 ? 0.f : Cvt<T>::to_f(reinterpret_cast<const T*>(a.cache_v)[(((long long)b * a.cap + ll_ring_row(p, a.keep, a.cap)) * a.G + g) * a.dvp + c]);
+      sV[x] = p < 0 ? 0.f : Cvt<T>::to_f(reinterpret_cast<const T*>(a.cache_v)[((long long)b * a.cap + ll_ring_row(p, a.keep, a.cap)) * a.ld_v + g * a.dvp + c]);
     }
     __syncthreads();
     const int kn = min(KT, kr.count - e0);
@@ -194,7 +212,7 @@ __global__ void __launch_bounds__(128) ll_attn_prefill_kernel(const __grid_const
         const int c = sub * 16 + d;
         if (c < a.dkp) s += q[d] * sK[kk * a.dkp + c];
       }
-      s = ll_group_sum<TPR>(s) * a.scale;
+      s = ll_score(ll_group_sum<TPR>(s), a.scale, a.softcap, slope, i - p);
       if (!live || p > i || !(a.window <= 0 || i - p < a.window || p < a.keep)) continue;
       const float mn = fmaxf(m, s);
       const float corr = expf(m - mn), pr = expf(s - mn);
@@ -215,7 +233,7 @@ __global__ void __launch_bounds__(128) ll_attn_prefill_kernel(const __grid_const
     l = l * fac + expf(sk - mn);
   }
   fac = l > 0.f ? fac / l : 0.f;
-  const T* gate = reinterpret_cast<const T*>(a.proj) + row * a.ld_proj + (a.H + a.G) * a.dk + a.G * a.dv + h * a.dv;
+  const T* gate = reinterpret_cast<const T*>(a.gate) + row * a.ld_gate + h * a.dv;
   T* op = reinterpret_cast<T*>(a.out) + row * a.ldo + h * a.dv;
 #pragma unroll
   for (int d = 0; d < 16; ++d) {
@@ -255,10 +273,11 @@ __global__ void __launch_bounds__(128) ll_attn_decode_kernel(const __grid_consta
   const int per = (kr.count + a.splits - 1) / a.splits;
   const int lo = split * per, hi = min(kr.count, lo + per);
   const bool kl = lane * EPL < a.dkp, vl = lane * EPL < a.dvp;
-  float q[GQ][EPL], o[GQ][EPL], m[GQ], l[GQ];
+  float q[GQ][EPL], o[GQ][EPL], m[GQ], l[GQ], slope[GQ];
 #pragma unroll
   for (int x = 0; x < GQ; ++x) {
     m[x] = -INFINITY; l[x] = 0.f;
+    slope[x] = a.slopes && x < nh ? a.slopes[h0 + x] : 0.f;
 #pragma unroll
     for (int e = 0; e < EPL; ++e) { q[x][e] = 0.f; o[x][e] = 0.f; }
     if (x < nh && kl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.q) + ((long long)b * a.H + h0 + x) * a.dkp + lane * EPL, q[x]);
@@ -266,15 +285,17 @@ __global__ void __launch_bounds__(128) ll_attn_decode_kernel(const __grid_consta
   constexpr int KB = EPL <= 4 ? 4 : 2;            // keys in flight per warp: all their loads come before the first use
   for (int e0 = lo + warp * KB; e0 < hi; e0 += 4 * KB) {
     float kf[KB][EPL], vf[KB][EPL];
+    int back[KB];
 #pragma unroll
     for (int j = 0; j < KB; ++j) {
       const int e = min(e0 + j, hi - 1);
       const int p = e < kr.n_kept ? e : kr.win_lo + (e - kr.n_kept);
-      const long long crow = ((long long)b * a.cap + ll_ring_row(p, a.keep, a.cap)) * a.G + g;
+      back[j] = pos - p;
+      const long long crow = (long long)b * a.cap + ll_ring_row(p, a.keep, a.cap);
 #pragma unroll
       for (int x = 0; x < EPL; ++x) { kf[j][x] = 0.f; vf[j][x] = 0.f; }
-      if (kl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.cache_k) + crow * a.dkp + lane * EPL, kf[j]);
-      if (vl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.cache_v) + crow * a.dvp + lane * EPL, vf[j]);
+      if (kl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.cache_k) + crow * a.ld_k + g * a.dkp + lane * EPL, kf[j]);
+      if (vl) ll_load<T, EPL>(reinterpret_cast<const T*>(a.cache_v) + crow * a.ld_v + g * a.dvp + lane * EPL, vf[j]);
     }
 #pragma unroll
     for (int x = 0; x < GQ; ++x) {
@@ -291,7 +312,7 @@ __global__ void __launch_bounds__(128) ll_attn_decode_kernel(const __grid_consta
         for (int j = 0; j < KB; ++j) s[j] += __shfl_xor_sync(0xffffffffu, s[j], d);
 #pragma unroll
       for (int j = 0; j < KB; ++j) {
-        s[j] = e0 + j < hi ? s[j] * a.scale : -INFINITY;
+        s[j] = e0 + j < hi ? ll_score(s[j], a.scale, a.softcap, slope[x], back[j]) : -INFINITY;
         mn = fmaxf(mn, s[j]);
       }
       const float c = expf(m[x] - mn);            // the first key of a group is always real, so mn is finite
@@ -358,7 +379,7 @@ __global__ void __launch_bounds__(128) ll_attn_merge_kernel(const __grid_constan
   float l = s_red[4] + s_red[5] + s_red[6] + s_red[7];
   if (a.sink) l += expf(a.sink[h] - mm);
   const float inv = l > 0.f ? 1.f / l : 0.f;
-  const T* gate = reinterpret_cast<const T*>(a.proj) + b * a.ld_proj + (a.H + a.G) * a.dk + a.G * a.dv + h * a.dv;
+  const T* gate = reinterpret_cast<const T*>(a.gate) + b * a.ld_gate + h * a.dv;
   T* op = reinterpret_cast<T*>(a.out) + b * a.ldo + h * a.dv;
   for (int c = tid; c < a.dv; c += 128) {
     float o = 0.f;
@@ -398,10 +419,10 @@ static int ll_prefill_go(const gb_ll_attn_args& a, cudaStream_t st) {
 using namespace gb;
 
 static int ll_attn_check(const gb_ll_attn_args* p) {
-  if (!p || !p->st || !p->proj || !p->q || !p->cache_k || !p->cache_v || p->B <= 0 || p->n <= 0 || p->G <= 0 || p->H <= 0 || p->H % p->G) return -1;
+  if (!p || !p->st || !p->q || !p->cache_k || !p->cache_v || p->B <= 0 || p->n <= 0 || p->G <= 0 || p->H <= 0 || p->H % p->G) return -1;
   if (p->dk <= 0 || p->dv <= 0 || p->dk > p->dkp || p->dv > p->dvp || p->dkp > 256 || p->dvp > 256 || p->dkp % 8 || p->dvp % 8) return -2;
   if (p->rot_dims < 0 || p->rot_dims % 2 || p->rot_dims > p->dk || (p->rot_dims > 0 && !p->freq)) return -3;
-  if (p->keep < 0 || p->cap <= p->keep || p->window < 0) return -4;
+  if (p->keep < 0 || p->cap <= p->keep || p->window < 0 || p->ld_k < p->G * p->dkp || p->ld_v < p->G * p->dvp || p->temp_every < 0) return -4;
   // the positions one call can see have to be in the ring together (window == 0: the caller bounds the length)
   if (p->window > 0 && p->pos0_max >= 0) {
     const long long last = (long long)p->pos0_max + p->n;
@@ -421,6 +442,7 @@ extern "C" int gb_ll_rotations(const double* freq, int pairs, const gb_seq_state
 
 extern "C" int gb_ll_qkv_store(const gb_ll_attn_args* p, cudaStream_t st) {
   if (const int rc = ll_attn_check(p)) return rc;
+  if (!p->proj || p->ld_k != p->G * p->dkp || p->ld_v != p->G * p->dvp) return -4;
   const long long items = (long long)p->B * p->n * (p->H + 2 * p->G);
   const bool vec = p->dk % 8 == 0 && p->dv % 8 == 0 && p->rot_dims % 8 == 0 && !p->rot_half && (p->cs || p->rot_dims == 0) && p->ld_proj % 8 == 0 &&
                    ((reinterpret_cast<uintptr_t>(p->proj) | reinterpret_cast<uintptr_t>(p->q) | reinterpret_cast<uintptr_t>(p->cache_k) |

@@ -6,6 +6,9 @@
 // from: an item's key tiles are the tiles of the kept prefix (rows 0 .. keep of the cache) followed by the ring tiles
 // that overlap its window.  The ring is a multiple of 128 rows long and starts at row `keep`, so a tile of 128
 // consecutive positions is 128 consecutive rows.  The item ends with the sink in the denominator and the output gate.
+//
+// CAPPED: scores pass through cap * tanh(. / cap), less slope * distance.  They are then at most cap, and at least -cap on
+// the query's own place, so exponentials need no running maximum: one pass over the scores, nothing to rescale.
 #include <algorithm>
 
 #include "sm100_common.cuh"
@@ -23,7 +26,15 @@ __device__ __forceinline__ float ll_ex2(float x) {
   return r;
 }
 
-template <int DK, int DV>
+constexpr float LA_CAP_MAX = 60.f;          // e^+-cap and sums of many such terms stay well inside fp32's range
+
+__device__ __forceinline__ float ll_rcp(float x) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+
+template <int DK, int DV, bool CAPPED>
 __global__ void __launch_bounds__(LA_THREADS) ll_attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ,
                                                                 const __grid_constant__ CUtensorMap tmK,
                                                                 const __grid_constant__ CUtensorMap tmV,
@@ -97,6 +108,10 @@ __global__ void __launch_bounds__(LA_THREADS) ll_attn_tc_kernel(const __grid_con
     return it.b * a.cap + (t < it.n_kt ? t * AT_N : a.keep + (int)(((long long)(it.r_lo + t - it.n_kt) * AT_N) % ring));
   };
 
+  auto tile_pos = [&](const Item& it, int t) {          // position of that row
+    return t < it.n_kt ? t * AT_N : a.keep + (it.r_lo + t - it.n_kt) * AT_N;
+  };
+
   if (warp == 4) {
     if (lane == 0) {
       uint32_t kv_it = 0, q_it = 0;
@@ -148,13 +163,16 @@ __global__ void __launch_bounds__(LA_THREADS) ll_attn_tc_kernel(const __grid_con
     const int r = threadIdx.x;
     const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
     const float sc2 = a.scale * 1.4426950408889634f;
+    // tanh(z) = 1 - 2 / (e^2z + 1): the exponent's factor, and cap in log2 units
+    const float cap_in = CAPPED ? 2.f * sc2 / a.softcap : 0.f, cap2 = a.softcap * 1.4426950408889634f;
     uint32_t tile_it = 0;
     bool ok = true;
     for (int item = blockIdx.x; item < n_items && ok; item += gridDim.x) {
       const Item it = item_of(item);
       const int i = it.p0 + it.q0 + r, i_first = it.p0 + it.q0, i_last = it.p0 + min(a.n, it.q0 + AT_M) - 1;
       const bool row_ok = it.q0 + r < a.n;
-      float m2 = -INFINITY, l = 0.f;            // maximum in use (log2 units) and the row sum against it
+      float m2 = CAPPED ? 0.f : -INFINITY, l = 0.f;            // maximum in use (log2 units) and the row sum against it
+      const float slope2 = CAPPED && a.slopes ? a.slopes[it.h] * 1.4426950408889634f : 0.f;
       for (int t = 0; t < it.n_kt + it.n_rt; ++t, ++tile_it) {
         // visible columns of this tile: lo .. hi
         int lo, hi;
@@ -171,55 +189,73 @@ __global__ void __launch_bounds__(LA_THREADS) ll_attn_tc_kernel(const __grid_con
         }
         if (!at_wait(s_full, tile_it & 1u, a.status, ST_TIMEOUT_TMEM_FULL, abort_flag)) { ok = false; break; }
         tc_fence_after();
-        float mr[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        if constexpr (!CAPPED) {
+          float mr[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll 1
-        for (int c = 0; c < AT_N / 32; ++c) {
-          uint32_t rg[32];
-          tmem_ld_32x32(tmem_S + lane_base + c * 32, rg);
-          tmem_ld_wait();
-          if (!need_mask) {
+          for (int c = 0; c < AT_N / 32; ++c) {
+            uint32_t rg[32];
+            tmem_ld_32x32(tmem_S + lane_base + c * 32, rg);
+            tmem_ld_wait();
+            if (!need_mask) {
 #pragma unroll
-            for (int k = 0; k < 32; ++k) mr[k & 3] = fmaxf(mr[k & 3], __uint_as_float(rg[k]));
-          } else {
+              for (int k = 0; k < 32; ++k) mr[k & 3] = fmaxf(mr[k & 3], __uint_as_float(rg[k]));
+            } else {
 #pragma unroll
-            for (int k = 0; k < 32; ++k) {
-              const int j = c * 32 + k;
-              if (j <= hi && j >= lo) mr[k & 3] = fmaxf(mr[k & 3], __uint_as_float(rg[k]));
+              for (int k = 0; k < 32; ++k) {
+                const int j = c * 32 + k;
+                if (j <= hi && j >= lo) mr[k & 3] = fmaxf(mr[k & 3], __uint_as_float(rg[k]));
+              }
             }
           }
-        }
-        float mt = fmaxf(fmaxf(mr[0], mr[1]), fmaxf(mr[2], mr[3])) * sc2;
-        if (!row_ok) mt = 0.f;
-        const bool grow = mt > m2 + 8.f || (m2 == -INFINITY && mt != -INFINITY);
-        if (__any_sync(0xffffffffu, grow)) {
-          const float m_new = fmaxf(m2, mt);
-          if (t > 0) {
-            const float corr = (m2 == -INFINITY) ? 1.f : ll_ex2(m2 - m_new);
-            l *= corr;
-            if (!at_wait(o_full, (tile_it - 1u) & 1u, a.status, ST_TIMEOUT_TMEM_FULL, abort_flag)) { ok = false; break; }
-            tc_fence_after();
+          float mt = fmaxf(fmaxf(mr[0], mr[1]), fmaxf(mr[2], mr[3])) * sc2;
+          if (!row_ok) mt = 0.f;
+          const bool grow = mt > m2 + 8.f || (m2 == -INFINITY && mt != -INFINITY);
+          if (__any_sync(0xffffffffu, grow)) {
+            const float m_new = fmaxf(m2, mt);
+            if (t > 0) {
+              const float corr = (m2 == -INFINITY) ? 1.f : ll_ex2(m2 - m_new);
+              l *= corr;
+              if (!at_wait(o_full, (tile_it - 1u) & 1u, a.status, ST_TIMEOUT_TMEM_FULL, abort_flag)) { ok = false; break; }
+              tc_fence_after();
 #pragma unroll
-            for (int c = 0; c < DV / 16; ++c) {
-              uint32_t rg[16];
-              tmem_ld_32x16(tmem_O + lane_base + c * 16, rg);
-              tmem_ld_wait();
+              for (int c = 0; c < DV / 16; ++c) {
+                uint32_t rg[16];
+                tmem_ld_32x16(tmem_O + lane_base + c * 16, rg);
+                tmem_ld_wait();
 #pragma unroll
-              for (int k = 0; k < 16; ++k) rg[k] = __float_as_uint(__uint_as_float(rg[k]) * corr);
-              tmem_st_32x16(tmem_O + lane_base + c * 16, rg);
+                for (int k = 0; k < 16; ++k) rg[k] = __float_as_uint(__uint_as_float(rg[k]) * corr);
+                tmem_st_32x16(tmem_O + lane_base + c * 16, rg);
+              }
+              tmem_st_wait();
             }
-            tmem_st_wait();
+            m2 = m_new;
           }
-          m2 = m_new;
         }
         float ls[2] = {0.f, 0.f};
         const bool dead = m2 == -INFINITY || !row_ok;
+        const float near2 = CAPPED ? cap2 - slope2 * (float)(i - tile_pos(it, t)) : 0.f;     // cap less the bias, at the tile's column 0
 #pragma unroll 1
         for (int c = 0; c < AT_N / 32; ++c) {
           uint32_t rg[32];
           tmem_ld_32x32(tmem_S + lane_base + c * 32, rg);
           tmem_ld_wait();
           float pv[32];
-          if (!need_mask) {
+          if constexpr (CAPPED) {
+            const float near_c = near2 + slope2 * (float)(c * 32);
+#pragma unroll
+            for (int k = 0; k < 32; ++k) {
+              const float th = ll_rcp(1.f + ll_ex2(__uint_as_float(rg[k]) * cap_in));
+              const float e = ll_ex2(fmaf(-2.f * cap2, th, fmaf(slope2, (float)k, near_c)));
+              pv[k] = e;
+            }
+            if (need_mask) {
+#pragma unroll
+              for (int k = 0; k < 32; ++k)
+                if (dead || c * 32 + k > hi || c * 32 + k < lo) pv[k] = 0.f;
+            }
+#pragma unroll
+            for (int k = 0; k < 32; ++k) ls[k & 1] += pv[k];
+          } else if (!need_mask) {
 #pragma unroll
             for (int k = 0; k < 32; ++k) {
               const float e = ll_ex2(fmaf(__uint_as_float(rg[k]), sc2, -m2));
@@ -255,7 +291,7 @@ __global__ void __launch_bounds__(LA_THREADS) ll_attn_tc_kernel(const __grid_con
       fac = l > 0.f ? fac / l : 0.f;
       const long long row = (long long)it.b * a.n + it.q0 + r;
       T* op = reinterpret_cast<T*>(a.out) + row * a.ldo + it.h * a.dv;
-      const T* gp = reinterpret_cast<const T*>(a.proj) + row * a.ld_proj + (a.H + a.G) * a.dk + a.G * a.dv + it.h * a.dv;
+      const T* gp = reinterpret_cast<const T*>(a.gate) + row * a.ld_gate + it.h * a.dv;
       const bool vec = a.dv == DV && ((reinterpret_cast<uintptr_t>(op) | reinterpret_cast<uintptr_t>(gp)) & 15) == 0;
 #pragma unroll
       for (int c = 0; c < DV / 32; ++c) {
@@ -307,16 +343,16 @@ __global__ void __launch_bounds__(LA_THREADS) ll_attn_tc_kernel(const __grid_con
   if (warp == 5) { tc_fence_after(); tmem_dealloc(tmem_base, 256); }
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool CAPPED>
 static int ll_attn_tc_go(const gb_ll_attn_args& a, cudaStream_t st) {
   CUtensorMap tq, tk, tv;
   const uint64_t rows = (uint64_t)a.B * a.n, crows = (uint64_t)a.B * a.cap;
   if (gb_make_tmap_2d_16b(&tq, a.q, rows, (uint64_t)a.H * DK, (uint64_t)a.H * DK, AT_M, 64, 1)) return -20;
-  if (gb_make_tmap_2d_16b(&tk, a.cache_k, crows, (uint64_t)a.G * DK, (uint64_t)a.G * DK, AT_N, 64, 1)) return -21;
-  if (gb_make_tmap_2d_16b(&tv, a.cache_v, crows, (uint64_t)a.G * DV, (uint64_t)a.G * DV, AT_N, 64, 1)) return -22;
+  if (gb_make_tmap_2d_16b(&tk, a.cache_k, crows, (uint64_t)a.G * DK, (uint64_t)a.ld_k, AT_N, 64, 1)) return -21;
+  if (gb_make_tmap_2d_16b(&tv, a.cache_v, crows, (uint64_t)a.G * DV, (uint64_t)a.ld_v, AT_N, 64, 1)) return -22;
   constexpr bool pair = DK == 64 && DV == 64;
   constexpr size_t smem = (size_t)AT_M * DK * 2 * 3 + (size_t)AT_N * DV * 2 * 2 + AT_M * AT_N * 2 + 128 + (pair ? 0 : 1024);
-  auto kern = ll_attn_tc_kernel<DK, DV>;
+  auto kern = ll_attn_tc_kernel<DK, DV, CAPPED>;
   static int sms = 0;
   if (!sms) {
     int dev = 0;
@@ -330,6 +366,12 @@ static int ll_attn_tc_go(const gb_ll_attn_args& a, cudaStream_t st) {
   return gb_launch_rc();
 }
 
+template <bool CAPPED>
+static int ll_attn_tc_sizes(const gb_ll_attn_args& a, cudaStream_t st) {
+  if (a.dkp == 64) return a.dvp == 64 ? ll_attn_tc_go<64, 64, CAPPED>(a, st) : ll_attn_tc_go<64, 128, CAPPED>(a, st);
+  return a.dvp == 64 ? ll_attn_tc_go<128, 64, CAPPED>(a, st) : ll_attn_tc_go<128, 128, CAPPED>(a, st);
+}
+
 }  // namespace gb
 
 using namespace gb;
@@ -337,7 +379,9 @@ using namespace gb;
 extern "C" int gb_ll_attn_tc_ok(const gb_ll_attn_args* p) {
   if (!p || p->dtype != 1) return -1;
   if ((p->dkp != 64 && p->dkp != 128) || (p->dvp != 64 && p->dvp != 128)) return -2;
-  if (!(p->scale > 0.f)) return -3;                       // the row maximum is taken on raw scores
+  if (p->softcap > 0.f ? p->softcap > LA_CAP_MAX : p->slopes != nullptr) return -3;
+  if (!(p->softcap > 0.f) && !(p->scale > 0.f)) return -3;          // the row maximum is taken on raw scores
+  if (p->ld_k % 8 || p->ld_v % 8 || p->ld_k < p->G * p->dkp || p->ld_v < p->G * p->dvp) return -4;
   if (p->cap <= p->keep || (p->cap - p->keep) % AT_N) return -4;
   if ((long long)p->B * p->cap > 0x7fffffffll || (long long)p->B * p->n > 0x7fffffffll) return -5;
   return 0;
@@ -345,7 +389,6 @@ extern "C" int gb_ll_attn_tc_ok(const gb_ll_attn_args* p) {
 
 extern "C" int gb_ll_attn_tc(const gb_ll_attn_args* p, cudaStream_t st) {
   if (const int rc = gb_ll_attn_tc_ok(p)) return rc;
-  if (!p->q || !p->cache_k || !p->cache_v || !p->proj || !p->out || !p->st || !p->status || p->B <= 0 || p->n <= 0 || p->H % p->G) return -1;
-  if (p->dkp == 64) return p->dvp == 64 ? ll_attn_tc_go<64, 64>(*p, st) : ll_attn_tc_go<64, 128>(*p, st);
-  return p->dvp == 64 ? ll_attn_tc_go<128, 64>(*p, st) : ll_attn_tc_go<128, 128>(*p, st);
+  if (!p->q || !p->cache_k || !p->cache_v || !p->out || !p->st || !p->status || p->B <= 0 || p->n <= 0 || p->H % p->G) return -1;
+  return p->softcap > 0.f ? ll_attn_tc_sizes<true>(*p, st) : ll_attn_tc_sizes<false>(*p, st);
 }

@@ -1,5 +1,6 @@
 // Row-wise kernels of layer-list models (interface in gb_layers.h): embedding, norms on sublayer outputs with the residual
-// add, the fp32 matrix product, the fp32 SwiGLU, the logit cap.
+// add, residual adds with the norm ahead of the next sublayer, the fp32 matrix product, the fp32 SwiGLU and squared
+// relu, the logit cap.
 #include <type_traits>
 
 #include "sm100_common.cuh"
@@ -90,6 +91,77 @@ __global__ void __launch_bounds__(256) ll_norm_rows_kernel(const float* __restri
   for (int i = lane; i < d; i += 32) ss += xr[i] * xr[i];
   const float inv = ll_inv_rms(warp_sum(ss), d, eps);
   for (int i = lane; i < ldo; i += 32) out[r * ldo + i] = Cvt<T>::from_f(i < d ? xr[i] * inv * w[i] : 0.f);
+}
+
+template <typename T, int TPR, int V>
+__global__ void __launch_bounds__(256) ll_embed_norm_kernel(const int* __restrict__ ids, const T* __restrict__ table, long long ld_table, int vocab,
+                                                            int mode, const float* __restrict__ w, const float* __restrict__ b, float eps,
+                                                            float* __restrict__ x, int rows, int d) {
+  pdl_wait();
+  __shared__ float red[8];
+  const int r = TPR == 32 ? blockIdx.x * 8 + (threadIdx.x >> 5) : blockIdx.x;
+  if (r >= rows) return;
+  const int id = ids[r];
+  const bool ok = id >= 0 && id < vocab;
+  auto get = [&](int i, float (&v)[V]) {
+    if (ok) ll_get(table + (long long)id * ld_table + i, v);
+    else {
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = 0.f;
+    }
+  };
+  ll_row_norm<TPR, V>(d, mode, w, b, eps, red, get, get, [&](int i, const float (&v)[V]) { ll_put(x + (long long)r * d + i, v); });
+}
+
+template <typename T, int TPR, int V>
+__global__ void __launch_bounds__(256) ll_add_norm_kernel(const float* __restrict__ y, long long ldy, float alpha, const float* x, const float* x0,
+                                                          const int* __restrict__ row_idx, int mode, const float* __restrict__ w,
+                                                          const float* __restrict__ b, float eps, float* x_out, T* __restrict__ out,
+                                                          long long ldo, int rows, int d) {
+  pdl_wait();
+  __shared__ float red[8];
+  const int r = TPR == 32 ? blockIdx.x * 8 + (threadIdx.x >> 5) : blockIdx.x;
+  if (r >= rows) return;
+  const long long src = (long long)(row_idx ? row_idx[r] : r) * d;
+  auto add = [&](int i, float (&v)[V]) {
+    ll_get(x + src + i, v);
+    if (y) {
+      float u[V];
+      ll_get(y + (long long)r * ldy + i, u);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] += alpha * u[e];
+    }
+    if (x0) {
+      float u[V];
+      ll_get(x0 + src + i, u);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] += u[e];
+    }
+  };
+  auto get = [&](int i, float (&v)[V]) {
+    add(i, v);
+    if (x_out) ll_put(x_out + (long long)r * d + i, v);
+  };
+  if (!out) {
+    for (int i = (threadIdx.x % TPR) * V; i < d; i += TPR * V) {
+      float v[V];
+      get(i, v);
+    }
+    return;
+  }
+  ll_row_norm<TPR, V>(d, mode, w, b, eps, red, get,
+                      [&](int i, float (&v)[V]) { if (x_out) ll_get(x_out + (long long)r * d + i, v); else add(i, v); },
+                      [&](int i, const float (&v)[V]) { ll_put(out + r * ldo + i, v); });
+  for (int i = d + threadIdx.x % TPR; i < ldo; i += TPR) out[r * ldo + i] = Cvt<T>::from_f(0.f);
+}
+
+__global__ void ll_relu2_kernel(float* __restrict__ v, long long ld, int n) {
+  pdl_wait();
+  float* row = v + blockIdx.y * ld;
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
+    const float a = fmaxf(row[i], 0.f);
+    row[i] = a * a;
+  }
 }
 
 __global__ void ll_softcap_kernel(float* __restrict__ v, long long ld, int n, float cap) {
@@ -195,6 +267,52 @@ extern "C" int gb_ll_norm_rows(const float* x, const int* row_idx, const float* 
   if (dtype == 1) GB_PDL_LAUNCH(ll_norm_rows_kernel<__nv_bfloat16>, grid, dim3(256), st, x, row_idx, w, eps, (__nv_bfloat16*)out, ldo, rows, d);
   else if (dtype == 2) GB_PDL_LAUNCH(ll_norm_rows_kernel<float>, grid, dim3(256), st, x, row_idx, w, eps, (float*)out, ldo, rows, d);
   else return -2;
+  return gb_launch_rc();
+}
+
+// a warp per row while the row fits its registers, else a block per row
+#define LL_ROWS(KERN, T, ...)                                                                                                 \
+  do {                                                                                                                       \
+    if (d <= 1024) {                                                                                                         \
+      if (vec) GB_PDL_LAUNCH((KERN<T, 32, 4>), dim3((rows + 7) / 8), dim3(256), st, __VA_ARGS__);                               \
+      else GB_PDL_LAUNCH((KERN<T, 32, 1>), dim3((rows + 7) / 8), dim3(256), st, __VA_ARGS__);                                   \
+    } else if (vec) GB_PDL_LAUNCH((KERN<T, 256, 4>), dim3(rows), dim3(256), st, __VA_ARGS__);                                   \
+    else GB_PDL_LAUNCH((KERN<T, 256, 1>), dim3(rows), dim3(256), st, __VA_ARGS__);                                              \
+  } while (0)
+
+static bool ll_norm_ok(int mode, const float* w) { return w && (mode == GB_LL_NORM_RMS || mode == GB_LL_NORM_LAYER); }
+static uintptr_t ll_bits(const void* p) { return reinterpret_cast<uintptr_t>(p); }
+
+extern "C" int gb_ll_embed_norm(const int* ids, const void* table, long long ld_table, int vocab, int mode, const float* w, const float* b,
+                                float eps, float* x, int rows, int d, int dtype, cudaStream_t st) {
+  if (!ids || !table || !x || rows <= 0 || d <= 0 || ld_table < d || vocab <= 0 || !ll_norm_ok(mode, w)) return -1;
+  const bool vec = d % 4 == 0 && ld_table % 4 == 0 && ((ll_bits(table) | ll_bits(x)) & 15) == 0;
+#define EN(T) LL_ROWS(ll_embed_norm_kernel, T, ids, (const T*)table, ld_table, vocab, mode, w, b, eps, x, rows, d)
+  if (dtype == 1) EN(__nv_bfloat16);
+  else if (dtype == 2) EN(float);
+  else return -2;
+#undef EN
+  return gb_launch_rc();
+}
+
+extern "C" int gb_ll_add_norm(const float* y, long long ldy, float alpha, const float* x, const float* x0, const int* row_idx, int mode,
+                              const float* w, const float* b, float eps, float* x_out, void* out, long long ldo, int rows, int d,
+                              int dtype, cudaStream_t st) {
+  if (!x || rows <= 0 || d <= 0 || (!x_out && !out) || (out && (!ll_norm_ok(mode, w) || ldo < d))) return -1;
+  if (row_idx && (y || x0 || x_out)) return -3;
+  const bool vec = d % 4 == 0 && (!y || ldy % 4 == 0) && (!out || ldo % 4 == 0) &&
+                   ((ll_bits(y) | ll_bits(x) | ll_bits(x0) | ll_bits(x_out) | ll_bits(out)) & 15) == 0;
+#define AN(T) LL_ROWS(ll_add_norm_kernel, T, y, ldy, alpha, x, x0, row_idx, mode, w, b, eps, x_out, (T*)out, ldo, rows, d)
+  if (dtype == 1) AN(__nv_bfloat16);
+  else if (dtype == 2) AN(float);
+  else return -2;
+#undef AN
+  return gb_launch_rc();
+}
+
+extern "C" int gb_ll_relu2_f32(float* v, long long ld, int rows, int n, cudaStream_t st) {
+  if (!v || rows <= 0 || n <= 0) return -1;
+  GB_PDL_LAUNCH(ll_relu2_kernel, dim3((n + 1023) / 1024, rows), dim3(256), st, v, ld, n);
   return gb_launch_rc();
 }
 

@@ -47,6 +47,8 @@ struct LlGemv {
   const void* y16; long long ldy16; const void* z16; long long ldz; int parts;
   const float* v32; const float* sq; int n_sq;
   void* out; long long ldo; int out_f32; float softcap;
+  const float* x0; float alpha; const float* b1; int norm_mode;
+  int n1; void* out2; long long ldo2;
 };
 
 // Input vector of sequence b into xs[0, K).
@@ -115,6 +117,51 @@ __device__ __forceinline__ void ll_prologue(const LlGemv& a, int b, XT* __restri
       const int i = tid + k * LV_THREADS;
       if (i < d) xs[i] = Cvt<XT>::from_f(v[k]);
     }
+  } else if constexpr (PRO == 4) {                 // weighted RMS norm of a 16-bit (fp32) vector
+    const XT* xr = reinterpret_cast<const XT*>(a.x16) + b * a.ldx;
+    float ss = 0.f;
+    for (int i = tid; i < d; i += LV_THREADS) { const float v = Cvt<XT>::to_f(xr[i]); ss += v * v; }
+    const float inv = ll_inv_rms(ll_block_sum(ss, red), d, a.eps);
+    for (int i = tid; i < d; i += LV_THREADS) xs[i] = Cvt<XT>::from_f(Cvt<XT>::to_f(xr[i]) * inv * a.w1[i]);
+  } else if constexpr (PRO == 5) {                 // residual add, then the norm ahead of the sublayers
+    const float* xr = a.x + (long long)b * d;
+    const float* yr = a.y ? a.y + b * a.ldy : nullptr;
+    const float* x0 = a.x0 ? a.x0 + (long long)b * d : nullptr;
+    float* xo = blockIdx.x == 0 && a.x_out ? a.x_out + (long long)b * d : nullptr;
+    constexpr int KEEP = 16;                       // values per thread kept in registers (d up to 4096); the rest is made again
+    auto value = [&](int i) {
+      float v = xr[i];
+      if (yr) v += a.alpha * yr[i];
+      if (x0) v += x0[i];
+      return v;
+    };
+    float v[KEEP];
+    float sum = 0.f, dev = 0.f;
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int i = tid + k * LV_THREADS;
+      v[k] = i < d ? value(i) : 0.f;
+      sum += v[k];
+    }
+    for (int i = tid + KEEP * LV_THREADS; i < d; i += LV_THREADS) sum += value(i);
+    const float mean = a.norm_mode == GB_LL_NORM_LAYER ? ll_block_sum(sum, red) / (float)d : 0.f;
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int i = tid + k * LV_THREADS;
+      if (i < d) { const float c = v[k] - mean; dev += c * c; }
+    }
+    for (int i = tid + KEEP * LV_THREADS; i < d; i += LV_THREADS) { const float c = value(i) - mean; dev += c * c; }
+    const float inv = ll_inv_rms(ll_block_sum(dev, red), d, a.eps);
+    auto put = [&](int i, float u) {
+      if (xo) xo[i] = u;
+      xs[i] = Cvt<XT>::from_f((u - mean) * inv * a.w1[i] + (a.b1 ? a.b1[i] : 0.f));
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int i = tid + k * LV_THREADS;
+      if (i < d) put(i, v[k]);
+    }
+    for (int i = tid + KEEP * LV_THREADS; i < d; i += LV_THREADS) put(i, value(i));
   } else if constexpr (PRO == 3) {                 // gated values and their sums of squares from the step kernel
     const float* vr = a.v32 + (long long)b * d;
     const float* sq = a.sq + (long long)b * a.n_sq;
@@ -298,7 +345,10 @@ __global__ void __launch_bounds__(LV_THREADS) ll_gemv_kernel(const __grid_consta
           if (k >= nb) continue;
           float v = SWI ? ll_silu(acc[k]) * acu[k] : acc[k];
           if (a.softcap > 0.f) v = a.softcap * tanhf(v / a.softcap);
-          if (a.out_f32) reinterpret_cast<float*>(a.out)[(long long)(b0 + k) * a.ldo + j] = v;
+          if (a.n1 > 0 && j >= a.n1) {
+            v = fmaxf(v, 0.f);
+            reinterpret_cast<XT*>(a.out2)[(long long)(b0 + k) * a.ldo2 + j - a.n1] = Cvt<XT>::from_f(v * v);
+          } else if (a.out_f32) reinterpret_cast<float*>(a.out)[(long long)(b0 + k) * a.ldo + j] = v;
           else reinterpret_cast<XT*>(a.out)[(long long)(b0 + k) * a.ldo + j] = Cvt<XT>::from_f(v);
         }
       }
@@ -338,6 +388,8 @@ static int ll_gemv_pro(const LlGemv& a, int prologue, int swiglu, cudaStream_t s
     case 1: return swiglu ? ll_gemv_go<FMT, XT, 1, 1>(a, st) : ll_gemv_go<FMT, XT, 1, 0>(a, st);
     case 2: return swiglu ? -1 : ll_gemv_go<FMT, XT, 2, 0>(a, st);
     case 3: return swiglu ? -1 : ll_gemv_go<FMT, XT, 3, 0>(a, st);
+    case 4: return swiglu ? -1 : ll_gemv_go<FMT, XT, 4, 0>(a, st);
+    case 5: return swiglu ? -1 : ll_gemv_go<FMT, XT, 5, 0>(a, st);
   }
   return -1;
 }
@@ -354,7 +406,12 @@ extern "C" int gb_ll_gemv(const gb_ll_gemv_args* p, cudaStream_t st) {
   if (p->prologue == 1 && (!p->x || (p->y && !p->w1) || (p->w2 && p->d > 4096))) return -1;
   if (p->prologue == 2 && (!p->y16 || !p->z16 || !p->w1 || p->parts <= 0 || p->d % p->parts)) return -1;
   if (p->prologue == 3 && (!p->v32 || !p->sq || !p->w1 || p->parts <= 0 || p->parts > 256 || p->d % p->parts || p->n_sq <= 0 || p->n_sq % p->parts)) return -1;
+  if (p->prologue == 4 && (!p->x16 || !p->w1)) return -1;
+  if (p->prologue == 5 && (!p->x || !p->w1 || (p->x_out && (p->x_out == p->x || p->x_out == p->x0)))) return -1;
+  if (p->n1 > 0 && (p->swiglu || !p->out2 || p->n1 > p->N)) return -1;
   LlGemv a{};
+  a.x0 = p->x0; a.alpha = p->alpha; a.b1 = p->b1; a.norm_mode = p->norm_mode;
+  a.n1 = p->n1; a.out2 = p->out2; a.ldo2 = p->ldo2;
   a.v32 = p->v32; a.sq = p->sq; a.n_sq = p->n_sq;
   a.W = static_cast<const uint8_t*>(p->W); a.row_bytes = rb; a.N = p->N; a.K = p->K; a.B = p->B; a.d = p->d;
   a.x16 = p->x16; a.ldx = p->ldx; a.x = p->x; a.y = p->y; a.ldy = p->ldy; a.w1 = p->w1; a.w2 = p->w2; a.eps = p->eps;

@@ -1,6 +1,7 @@
 // Small helpers shared by the kernels of layer-list models.
 #pragma once
 #include "sm100_common.cuh"
+#include "gb_layers.h"
 
 namespace gb {
 
@@ -64,6 +65,104 @@ __device__ __forceinline__ void ll_store4(__nv_bfloat16* p, const float4& v) {
   q.x = Cvt<__nv_bfloat16>::pack2(v.x, v.y);
   q.y = Cvt<__nv_bfloat16>::pack2(v.z, v.w);
   *reinterpret_cast<uint2*>(p) = q;
+}
+
+// V neighbouring values
+__device__ __forceinline__ void ll_get(const float* p, float (&v)[4]) {
+  const float4 q = *reinterpret_cast<const float4*>(p);
+  v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+}
+__device__ __forceinline__ void ll_get(const __nv_bfloat16* p, float (&v)[4]) {
+  LlRaw4<__nv_bfloat16> r;
+  r.load(p);
+  r.expand(v);
+}
+template <typename T> __device__ __forceinline__ void ll_get(const T* p, float (&v)[8]) { ll_load8(p, v); }
+template <typename T> __device__ __forceinline__ void ll_get(const T* p, float (&v)[1]) { v[0] = Cvt<T>::to_f(*p); }
+template <typename T> __device__ __forceinline__ void ll_put(T* p, const float (&v)[4]) { ll_store4(p, make_float4(v[0], v[1], v[2], v[3])); }
+template <typename T> __device__ __forceinline__ void ll_put(T* p, const float (&v)[8]) { ll_store8(p, v); }
+template <typename T> __device__ __forceinline__ void ll_put(T* p, const float (&v)[1]) { *p = Cvt<T>::from_f(v[0]); }
+
+// sum over the TPR threads of a row (a warp, or the block of 256); every thread gets it
+template <int TPR>
+__device__ __forceinline__ float ll_row_sum(float v, float* red) {
+  v = warp_sum(v);
+  if constexpr (TPR > 32) {
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    v = 0.f;
+#pragma unroll
+    for (int i = 0; i < TPR / 32; ++i) v += red[i];
+  }
+  return v;
+}
+
+// Norm of one row by TPR threads, V neighbouring values at a time.  `get(i, v)` gives the values at i .. i + V - 1 and is
+// called once per place, except for places past the ones kept in registers, which `again(i, v)` gives once more; `put(i, v)`
+// takes the normed values.
+template <int TPR, int V, typename Get, typename Again, typename Put>
+__device__ __forceinline__ void ll_row_norm(int d, int mode, const float* __restrict__ w, const float* __restrict__ b, float eps, float* red,
+                                            Get get, Again again, Put put) {
+  constexpr int KEEP = 8;
+  const int t = threadIdx.x % TPR;
+  float keep[KEEP][V];
+  float sum = 0.f, dev = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = (t + k * TPR) * V;
+    if (i < d) get(i, keep[k]);
+    else {
+#pragma unroll
+      for (int e = 0; e < V; ++e) keep[k][e] = 0.f;
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) sum += keep[k][e];
+  }
+  for (int i = (t + KEEP * TPR) * V; i < d; i += TPR * V) {
+    float v[V];
+    get(i, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) sum += v[e];
+  }
+  const float mean = mode == GB_LL_NORM_LAYER ? ll_row_sum<TPR>(sum, red) / (float)d : 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k)
+    if ((t + k * TPR) * V < d) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) { const float c = keep[k][e] - mean; dev += c * c; }
+    }
+  for (int i = (t + KEEP * TPR) * V; i < d; i += TPR * V) {
+    float v[V];
+    again(i, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) { const float c = v[e] - mean; dev += c * c; }
+  }
+  const float inv = ll_inv_rms(ll_row_sum<TPR>(dev, red), d, eps);
+  auto finish = [&](int i, float (&v)[V]) {
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = (v[e] - mean) * inv;
+    float u[V];
+    ll_get(w + i, u);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] *= u[e];
+    if (b) {
+      ll_get(b + i, u);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] += u[e];
+    }
+    put(i, v);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = (t + k * TPR) * V;
+    if (i < d) finish(i, keep[k]);
+  }
+  for (int i = (t + KEEP * TPR) * V; i < d; i += TPR * V) {
+    float v[V];
+    again(i, v);
+    finish(i, v);
+  }
 }
 
 // Cache row of a position: the first `keep` rows are never given up, the rest is a ring of cap - keep rows.

@@ -1,5 +1,6 @@
-"""Per-sequence memory of a layer-list model: one key/value cache per attention layer and one recurrent state per state-space
-layer (a layer that shares another layer's weights still has its own), for a fixed number of sequence slots.
+"""Per-sequence memory of a layer-list model: one key/value cache per attention layer, one cache of latents per latent-attention
+layer and one recurrent state per state-space layer (a layer that shares another layer's weights still has its own, a layer
+that runs several times has one per run), for a fixed number of sequence slots.
 
 An attention layer that only sees a window keeps ``keep_first + ring`` rows per sequence, with the ring long enough for
 the window plus one portion of a prompt; the row of a position is fixed (``gb_layers.h``), so nothing is moved and the
@@ -13,7 +14,8 @@ from typing import Dict, Hashable, List, Optional
 
 import torch
 
-from ..models.layer_list import AttentionMixer, LayerListConfig, Mamba2Mixer
+from ..models.layer_list import AttentionMixer, LatentAttentionMixer, LayerListConfig, Mamba2Mixer
+from ..ops.layers import head_pad
 from ..utils import canary as CA
 
 RING_ALIGN = 128          # key tiles of the tensor-core attention do not cross the end of the ring
@@ -21,11 +23,6 @@ RING_ALIGN = 128          # key tiles of the tensor-core attention do not cross 
 
 def _up(n: int, a: int) -> int:
     return (n + a - 1) // a * a
-
-
-def head_pad(d: int, dtype) -> int:
-    """Row length of a head in q and the caches (zero-padded): whole 128-byte panels for the tensor cores."""
-    return _up(d, 64) if dtype == torch.bfloat16 else _up(d, 8)
 
 
 class AttentionCache:
@@ -46,6 +43,18 @@ class AttentionCache:
         return (self.k.numel() + self.v.numel()) * self.k.element_size()
 
 
+class LatentCache:
+    """One row per token: the normed latent, then the rotated key part of all heads."""
+
+    def __init__(self, m: LatentAttentionMixer, slots: int, max_len: int, chunk: int, dtype, device):
+        self.cap = self.limit = _up(max_len, RING_ALIGN)
+        self.rows = CA.zeros(slots, self.cap, _up(m.kv_rank + m.rot_dim, 8), dtype=dtype, device=device)
+
+    @property
+    def nbytes(self):
+        return self.rows.numel() * self.rows.element_size()
+
+
 class RecurrentState:
     limit = None
 
@@ -59,14 +68,15 @@ class RecurrentState:
         return self.conv.numel() * self.conv.element_size() + self.ssm.numel() * 4
 
 
-KINDS = {AttentionMixer: AttentionCache, Mamba2Mixer: RecurrentState}
+KINDS = {AttentionMixer: AttentionCache, LatentAttentionMixer: LatentCache, Mamba2Mixer: RecurrentState}
 
 
 class SlotManager:
     """Layer memories plus the book of which request holds which slot and how many tokens it has seen."""
 
     def __init__(self, cfg: LayerListConfig, slots: int, max_len: int, chunk: int, dtype, device):
-        self.layers = [KINDS[type(s.mixer)](s.mixer, slots, max_len, chunk, dtype, device) for s in cfg.layers]
+        mixers = [cfg.layers[r.layer].mixer for r in cfg.runs]
+        self.layers = [KINDS[type(m)](m, slots, max_len, chunk, dtype, device) for m in mixers]      # by run
         limits = [c.limit for c in self.layers if c.limit is not None]
         self.limit: Optional[int] = min(limits) if limits else None       # most tokens a sequence may have (None: any)
         self.length: List[int] = [0] * slots

@@ -2,7 +2,7 @@
 
 A file or folder is turned into a configuration object, and the configuration decides the engine that serves it.  GGUF,
 legacy and checkpoint files hold the MoE / dense decoder of ``models/config.py``; a folder with ``config.json`` names its
-architecture, which is looked up here.  A further design made of known layer types is one more entry.
+architecture, which is looked up here.  A further design made of known layer types is one more entry (of ``DESIGNS`` in ``models/layer_list.py``).
 """
 from __future__ import annotations
 
@@ -10,7 +10,7 @@ from dataclasses import dataclass
 from typing import Callable, Dict
 
 from .config import ModelConfig
-from .layer_list import LayerListConfig
+from .layer_list import DESIGNS, LayerListConfig
 
 
 @dataclass(frozen=True)
@@ -29,7 +29,8 @@ def register(a: Architecture) -> Architecture:
     return a
 
 
-register(Architecture("Zikedra", LayerListConfig, LayerListConfig.from_json, "inference.layer_engine:LayerEngine"))
+for _name in DESIGNS:
+    register(Architecture(_name, LayerListConfig, LayerListConfig.from_json, "inference.layer_engine:LayerEngine"))
 
 
 def from_json(d: dict) -> Architecture:

@@ -14,7 +14,7 @@ import torch
 
 from . import _lib
 
-EPI_STORE, EPI_SWIGLU_FWD, EPI_SWIGLU_BWD = 0, 1, 2
+EPI_STORE, EPI_SWIGLU_FWD, EPI_SWIGLU_BWD, EPI_RELU2 = 0, 1, 2, 4
 
 # Two-CTA 256 x 256 tiles (csrc/cuda/gemm_pair_sm100.cu) are taken when the problem has at least this many of them
 # (74 CTA pairs on a B200); GB200_GEMM_PAIR=0 keeps every product on the one-CTA kernel.
@@ -85,8 +85,9 @@ def pick_block_n(M, N, mn_major=False):
     return 128
 
 
-def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_dtype=None, addend=None, block_n=0, pair=None):
+def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_dtype=None, addend=None, block_n=0, pair=None, relu2=False):
     """``out = A @ B^T (+ addend)``; ``addend`` is fp32 and may alias an fp32 ``out`` (accumulate).
+    ``relu2``: store ``max(A @ B^T, 0) ** 2`` (bf16, no addend).
     ``pair``: force (True) or forbid (False) the two-CTA kernel; None picks by size."""
     M, K = (a.shape[1], a.shape[0]) if a_mn else (a.shape[0], a.shape[1])
     N, Kb = (b.shape[1], b.shape[0]) if b_mn else (b.shape[0], b.shape[1])
@@ -99,7 +100,9 @@ def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_dtype=None, addend=None,
     if not block_n:
         block_n = pick_block_n(M, N, mn_major=a_mn and b_mn)
     g = _base_args(a, b, M, N, K, a_mn, b_mn, out, block_n)
-    g.epilogue = EPI_STORE
+    if relu2 and (addend is not None or out.dtype != torch.bfloat16):
+        raise ValueError("relu2 needs a bf16 output and no addend")
+    g.epilogue = EPI_RELU2 if relu2 else EPI_STORE
     g.pair = int(bool(pair))
     if addend is not None:
         if addend.dtype != torch.float32:

@@ -16,6 +16,12 @@ GEMV_MAX_SMEM = 200 * 1024
 FINAL_NORM_MAX = 4096                                # widest row whose last norm the GEMV prologue takes along
 
 
+def head_pad(d: int, dtype) -> int:
+    """Row length of a head in q and the caches (zero-padded): whole 128-byte panels for the tensor cores."""
+    a = 64 if dtype == torch.bfloat16 else 8
+    return (d + a - 1) // a * a
+
+
 class GemvArgs(ctypes.Structure):
     _fields_ = [
         ("W", c_vp), ("fmt", c_int), ("N", c_int), ("K", c_int),
@@ -25,6 +31,8 @@ class GemvArgs(ctypes.Structure):
         ("y16", c_vp), ("ldy16", c_ll), ("z16", c_vp), ("ldz", c_ll), ("parts", c_int),
         ("v32", c_vp), ("sq", c_vp), ("n_sq", c_int),
         ("out", c_vp), ("ldo", c_ll), ("out_f32", c_int), ("softcap", c_float),
+        ("x0", c_vp), ("alpha", c_float), ("b1", c_vp), ("norm_mode", c_int),
+        ("n1", c_int), ("out2", c_vp), ("ldo2", c_ll),
     ]
 
 
@@ -34,9 +42,24 @@ class AttnArgs(ctypes.Structure):
         ("dk", c_int), ("dv", c_int), ("dkp", c_int), ("dvp", c_int),
         ("rot_dims", c_int), ("rot_half", c_int), ("freq", c_vp), ("cs", c_vp), ("qk_norm", c_int), ("eps", c_float), ("scale", c_float),
         ("window", c_int), ("keep", c_int), ("cap", c_int),
-        ("proj", c_vp), ("ld_proj", c_ll), ("gate", c_int), ("sink", c_vp),
-        ("q", c_vp), ("cache_k", c_vp), ("cache_v", c_vp), ("out", c_vp), ("ldo", c_ll),
+        ("proj", c_vp), ("ld_proj", c_ll), ("gate", c_vp), ("ld_gate", c_ll), ("sink", c_vp),
+        ("softcap", c_float), ("slopes", c_vp), ("temp_coef", c_float), ("temp_every", c_int),
+        ("q", c_vp), ("cache_k", c_vp), ("cache_v", c_vp), ("ld_k", c_ll), ("ld_v", c_ll), ("out", c_vp), ("ldo", c_ll),
         ("scratch", c_vp), ("splits", c_int), ("st", c_vp), ("pos0_max", c_int), ("status", c_vp),
+    ]
+
+
+class LatentArgs(ctypes.Structure):
+    _fields_ = [
+        ("dtype", c_int), ("B", c_int), ("n", c_int),
+        ("H", c_int), ("dn", c_int), ("dr", c_int), ("dv", c_int), ("rank", c_int), ("q_rank", c_int),
+        ("dkp", c_int), ("dvp", c_int), ("rot_dims", c_int),
+        ("cs", c_vp), ("eps", c_float), ("scale", c_float),
+        ("proj", c_vp), ("ld_proj", c_ll), ("q_norm", c_vp), ("kv_norm", c_vp),
+        ("cq", c_vp), ("ld_cq", c_ll), ("cache", c_vp), ("ldc", c_int), ("cap", c_int),
+        ("qc", c_vp), ("ld_qc", c_ll), ("q", c_vp), ("W_kv", c_vp), ("ld_w", c_ll), ("qa", c_vp),
+        ("gate", c_vp), ("ld_gate", c_ll), ("out", c_vp), ("ldo", c_ll),
+        ("scratch", c_vp), ("splits", c_int), ("st", c_vp), ("status", c_vp),
     ]
 
 
@@ -75,6 +98,28 @@ def postnorm(y, x, w, eps, x_out, x16, rows, d):
 def norm_rows(x, row_idx, w, eps, out, rows, d):
     _call("gb_ll_norm_rows", _p(x), _p(row_idx), _p(w), c_float(eps), _p(out), c_ll(out.stride(0)), c_int(rows), c_int(d),
           c_int(DTYPE[out.dtype]))
+
+
+NORM = {"rms": 0, "layer": 1}
+
+
+def embed_norm(ids, table, norm, eps, x, dtype):
+    """``x = norm(table[ids])``; ``norm``: (kind, weight, bias or None)."""
+    kind, w, b = norm
+    _call("gb_ll_embed_norm", _p(ids), _p(table), c_ll(table.stride(0)), c_int(table.shape[0]), c_int(NORM[kind]), _p(w), _p(b), c_float(eps),
+          _p(x), c_int(ids.numel()), c_int(x.shape[1]), c_int(DTYPE[dtype]))
+
+
+def add_norm(x, rows, norm=None, eps=0.0, out=None, y=None, alpha=1.0, x0=None, x_out=None, row_idx=None):
+    """``v = x + alpha * y + x0``; ``x_out = v`` and ``out = norm(v)`` in the compute type, each where it is asked for."""
+    kind, w, b = norm if norm is not None else ("rms", None, None)
+    _call("gb_ll_add_norm", _p(y), c_ll(0 if y is None else y.stride(0)), c_float(alpha), _p(x), _p(x0), _p(row_idx), c_int(NORM[kind]), _p(w), _p(b),
+          c_float(eps), _p(x_out), _p(out), c_ll(0 if out is None else out.stride(0)), c_int(rows), c_int(x.shape[1]),
+          c_int(1 if out is None else DTYPE[out.dtype]))
+
+
+def relu2_f32(v, rows, n):
+    _call("gb_ll_relu2_f32", _p(v), c_ll(v.stride(0)), c_int(rows), c_int(n))
 
 
 def softcap(v, rows, n, cap):
@@ -122,6 +167,22 @@ def attn_tc(a: AttnArgs):
 
 def attn_decode(a: AttnArgs):
     _call("gb_ll_attn_decode", ctypes.byref(a))
+
+
+def latent_store(a: LatentArgs):
+    _call("gb_ll_latent_store", ctypes.byref(a))
+
+
+def latent_queries(a: LatentArgs):
+    _call("gb_ll_latent_queries", ctypes.byref(a))
+
+
+def latent_absorb(a: LatentArgs, store: bool):
+    _call("gb_ll_latent_absorb", ctypes.byref(a), c_int(int(store)))
+
+
+def latent_attn(a: LatentArgs):
+    _call("gb_ll_latent_attn", ctypes.byref(a))
 
 
 def conv(a: MambaArgs):

@@ -1,5 +1,6 @@
-"""Plain implementation of layer-list models (attention and Mamba-2 mixers, dense feed-forwards): the oracle of
-``tests/test_layers_*.py``.
+"""Plain implementation of layer-list models (attention, latent attention and Mamba-2 mixers, dense feed-forwards; layers in
+sequence or sublayers side by side, with repeated runs of layers): the oracle of ``tests/test_layers_*.py`` and
+``tests/test_parallel_*.py``.
 
 One function per mechanism, written from the equations in double precision, over whole sequences, with the recurrence
 as a loop over tokens.  It shares no code with the package: it takes the parsed JSON configuration and a dictionary of
@@ -152,6 +153,8 @@ def sub(w, prefix):
 def run(cfg, weights, tokens, want_layers=False):
     """Logits [tokens, vocab] of one sequence (and the residual after every layer)."""
     w = {k: np.asarray(v, dtype=np.float64) for k, v in weights.items()}
+    if cfg["architecture"] == "Dunavik":
+        return run_side_by_side(cfg, w, tokens, want_layers)
     eps = cfg["norm"]["eps"]
     x = w["embed"][np.asarray(tokens)]
     seen = []
@@ -164,4 +167,102 @@ def run(cfg, weights, tokens, want_layers=False):
     logits = (rms(x, eps) * w["final.norm"]) @ w["head"].T
     cap = cfg["logit_softcap"]
     logits = cap * np.tanh(logits / cap)
+    return (logits, seen) if want_layers else logits
+
+
+# ------------------------------------------------------------------------------------------------ side by side (Dunavik)
+def layer_norm(x, weight, bias, eps):
+    """Centred over the last axis, over the root of the mean squared deviation, scaled and shifted."""
+    c = x - x.mean(-1, keepdims=True)
+    return c / np.sqrt((c * c).mean(-1, keepdims=True) + eps) * weight + bias
+
+
+def softmax(scores, allowed):
+    s = np.where(allowed, scores, -np.inf)
+    e = np.exp(s - s.max(-1, keepdims=True))
+    return e / e.sum(-1, keepdims=True)
+
+
+def query_temperature(positions, coef, every):
+    """Factor of the query at each position: grows with the logarithm of the number of whole stretches behind it."""
+    return np.array([1.0 + coef * math.log((p + 1) // every + 1) for p in positions])
+
+
+def soft_cap(s, cap):
+    return cap * np.tanh(s / cap)
+
+
+def distance_slopes(heads):
+    return np.array([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)])
+
+
+def biased_attention(h, mix, w, eps):
+    """Sliding-window attention without rotation: tempered queries, capped scores less a slope times the distance."""
+    T = h.shape[0]
+    H, G, dk, dv = mix["heads"], mix["kv_heads"], mix["dim"], mix["vdim"]
+    q = (h @ w["q"].T).reshape(T, H, dk)
+    k = (h @ w["k"].T).reshape(T, G, dk)
+    v = (h @ w["v"].T).reshape(T, G, dv)
+    q = q * query_temperature(range(T), mix["q_temp"]["coef"], mix["q_temp"]["every"])[:, None, None]
+    back = np.arange(T)[:, None] - np.arange(T)[None, :]
+    see = (back >= 0) & (back < mix["mask"]["size"])
+    slopes = distance_slopes(H)
+    out = np.zeros((T, H, dv))
+    for a in range(H):
+        g = a // (H // G)
+        s = soft_cap((q[:, a] @ k[:, g].T) * mix["scale"], mix["softcap"]) - slopes[a] * back
+        out[:, a] = softmax(s, see) @ v[:, g]
+    return out.reshape(T, H * dv) @ w["o"].T
+
+
+def latent_attention(h, mix, w, eps):
+    """Queries from a normed latent; keys and values from another one, plus one rotated key part that all heads share."""
+    T = h.shape[0]
+    H, dn, dr, dv, R = mix["heads"], mix["dim"], mix["rot_dim"], mix["vdim"], mix["kv_rank"]
+    pos = np.arange(T)
+    q = ((rms(h @ w["dq"].T, eps) * w["dq.norm"]) @ w["uq"].T).reshape(T, H, dn + dr)
+    down = h @ w["dkv"].T
+    c = rms(down[:, :R], eps) * w["dkv.norm"]
+    k_rot = rotate(down[:, None, R:], mix["rot"], pos)[:, 0]
+    q_rot = rotate(q[:, :, dn:], mix["rot"], pos)
+    k = (c @ w["uk"].T).reshape(T, H, dn)
+    v = (c @ w["uv"].T).reshape(T, H, dv)
+    see = pos[None, :] <= pos[:, None]
+    out = np.zeros((T, H, dv))
+    for a in range(H):
+        s = (q[:, a, :dn] @ k[:, a].T + q_rot[:, a] @ k_rot.T) * mix["scale"]
+        out[:, a] = softmax(s, see) @ v[:, a]
+    return (out.reshape(T, H * dv) * sigmoid(h @ w["g"].T)) @ w["o"].T
+
+
+def squared_relu_mlp(h, w):
+    return np.square(np.maximum(h @ w["up"].T, 0.0)) @ w["down"].T
+
+
+def layer_runs(cfg):
+    """Layers in the order in which they run, with True where the embedding output joins before one."""
+    n, loop = len(cfg["layers"]), cfg.get("loop")
+    if not loop:
+        return [(i, False) for i in range(n)]
+    a, b = loop["start"], loop["stop"]
+    turns = [(i, t > 0 and i == a) for t in range(loop["times"]) for i in range(a, b)]
+    return [(i, False) for i in range(a)] + turns + [(i, False) for i in range(b, n)]
+
+
+def run_side_by_side(cfg, w, tokens, want_layers=False):
+    eps, mult = cfg["norm"]["eps"], cfg["residual_mult"]
+    mixers = {"attention": biased_attention, "latent_attention": latent_attention}
+    x = first = layer_norm(w["embed"][np.asarray(tokens)], w["embed.norm"], w["embed.norm.b"], eps)
+    seen = []
+    for i, rejoin in layer_runs(cfg):
+        p, layer = "l%d." % i, cfg["layers"][i]
+        if rejoin:
+            x = x + first
+        h = layer_norm(x, w[p + "norm1"], w[p + "norm1.b"], eps)
+        y = mixers[layer["type"]](h, layer["mixer"], sub(w, p + "mix."), eps)
+        if layer["mlp"] is not None:
+            y = y + squared_relu_mlp(h, sub(w, p + "mlp."))
+        x = x + mult * y
+        seen.append(x)
+    logits = layer_norm(x, w["final.norm"], w["final.norm.b"], eps) @ w["head"].T
     return (logits, seen) if want_layers else logits

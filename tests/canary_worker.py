@@ -86,13 +86,16 @@ training:
         torch.cuda.synchronize()
         bad += ["decode/%s/%s" % (kw, b) for b in CA.check()]
     # layer-list models: prompt passes, portions, both token steps, in both precisions
+    import dunavik_cases as DC
     import layers_cases as LC
     from ghassan_b200.inference.layer_engine import LayerEngine
     from ghassan_b200.models.layer_list import LayerListConfig
-    for name, raw in sorted(LC.cases().items()):
+    models = [(name, raw, LC.weights(raw)) for name, raw in sorted(LC.cases().items())]
+    models += [("dunavik " + name, raw, DC.weights(raw)) for name, raw in sorted(DC.cases().items())]
+    for name, raw, weights in models:
         for dtype in (torch.bfloat16, torch.float32):
             for B in (1, 9):
-                eng = LayerEngine(LayerListConfig.from_json(raw), LC.weights(raw), batch=B, max_len=400, prefill_chunk=70, dtype=dtype)
+                eng = LayerEngine(LayerListConfig.from_json(raw), weights, batch=B, max_len=400, prefill_chunk=70, dtype=dtype)
                 eng.reset(1)
                 eng.prefill(torch.tensor([LC.tokens(raw, 151, b) for b in range(B)], dtype=torch.int32))
                 sp = SamplingParams(seed=3, top_k=20)

@@ -1,6 +1,6 @@
 """Plain implementation of layer-list models (attention, latent attention and Mamba-2 mixers, dense feed-forwards; layers in
 sequence or sublayers side by side, with repeated runs of layers): the oracle of ``tests/test_layers_*.py`` and
-``tests/test_parallel_*.py``.
+``tests/test_dunavik_*.py``.
 
 One function per mechanism, written from the equations in double precision, over whole sequences, with the recurrence
 as a loop over tokens.  It shares no code with the package: it takes the parsed JSON configuration and a dictionary of

@@ -5,7 +5,7 @@ uniform token data, random-initialised weights.
     python bench.py --gpus N --steps K --warmup W                  # this framework
     python bench.py --impl reference --gpus N --steps K --warmup W  # the unmodified reference binary
     python bench.py --profile-passes 2 [--fuse F] [--layers L] [--end-step]   # a few eager passes, for use under ncu
-    python bench.py --layer-list [--sizes s,m,l]                    # layer-list models, kernels and throughput
+    python bench.py --layer-list [--design zikedra|dunavik] [--sizes s,m,l]   # layer-list models, kernels and throughput
     python bench.py --sync-only                                     # the gradient exchange alone (one process per GPU)
 
 With one GPU the JSON line also carries a ``decode`` object: batch-1 decode tokens/s of the same model for f16, q8_0 and
@@ -624,7 +624,7 @@ def main():
     ap.add_argument("--nvls", action="store_true", help="--sync-only: reduce and distribute through NVSwitch multicast")
     ap.add_argument("--sync-elements", type=int, default=1_036_995_840)
     ap.add_argument("--layer-list", nargs=argparse.REMAINDER, metavar="ARG",
-                    help="layer-list models (attention + Mamba-2) beside the dense decoder; what follows goes to bench_layers.py")
+                    help="layer-list models (attention + Mamba-2, or window + latent attention) beside the dense decoder; what follows goes to bench_layers.py")
     args = ap.parse_args()
     if args.layer_list is not None:
         import bench_layers

@@ -134,16 +134,20 @@ typedef struct gb_ll_latent_args {
   const void* qc; long long ld_qc;       // [rows, H, dn + dr] queries as projected
   void* q;                               // [rows, H, dkp] rotated queries
   const void* W_kv; long long ld_w;      // rows h*dkp + d: key map of head h, rows H*dkp + h*dvp + e: its value map; columns: rank ..
-  float* qa;                             // [rows, H, ldc] queries against cache rows
+  float* qa;                             // [rows, H, ldc] queries against cache rows, or
+  void* qa16; int heads_pad, ld_qa16;    // [rows, heads_pad, ld_qa16] the same in bf16 for the tensor cores (padding is zero)
   const void* gate; long long ld_gate;   // [rows, H*dv] or NULL
   void* out; long long ldo;              // [rows, H*dv]
-  float* scratch; int splits;            // rows * H * splits * (ldc + 2) floats
+  float* scratch; int splits;            // rows * H * splits * (ldc + 2) floats: partial outputs [.., ldc], then (maximum, sum)
   const gb_seq_state* st; int* status;
 } gb_ll_latent_args;
 int gb_ll_latent_store(const gb_ll_latent_args* a, cudaStream_t st);    // norms, rotation of k_rot: cq and the cache rows
 int gb_ll_latent_queries(const gb_ll_latent_args* a, cudaStream_t st);  // q = qc with its rotated part turned, padded
-int gb_ll_latent_absorb(const gb_ll_latent_args* a, int store, cudaStream_t st);   // qa; store != 0: the cache rows, too
-int gb_ll_latent_attn(const gb_ll_latent_args* a, cudaStream_t st);     // rank + dr up to 1024
+int gb_ll_latent_absorb(const gb_ll_latent_args* a, int store, cudaStream_t st);   // qa or qa16; store != 0: the cache rows, too
+int gb_ll_latent_attn(const gb_ll_latent_args* a, cudaStream_t st);     // rank + dr up to 1024; on the tensor cores with qa16
+// 0 when the tensor-core kernel covers the shapes (bf16, cap a multiple of 128): heads_pad and ld_qa16 to use.
+int gb_ll_latent_tc_plan(const gb_ll_latent_args* a, int* heads_pad, int* ld_qa16);
+int gb_ll_latent_tc(const gb_ll_latent_args* a, cudaStream_t st);       // the part of gb_ll_latent_attn before the merge
 
 // ------------------------------------------------------------------------------------------------ Mamba-2
 typedef struct gb_ll_mamba_args {

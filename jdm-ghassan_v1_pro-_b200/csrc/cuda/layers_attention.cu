@@ -23,9 +23,11 @@ __device__ __forceinline__ float ll_query_temperature(int pos, float coef, int e
 }
 
 // Score as the soft-max sees it: scaled, capped, less the slope times the distance.
+// (T of 16 bits: tanh(z) = 1 - 2 / (e^2z + 1) with the hardware's exponential and quotient, about 1e-6 of the cap.)
+template <typename T>
 __device__ __forceinline__ float ll_score(float dot, float scale, float cap, float slope, int back) {
   float s = dot * scale;
-  if (cap > 0.f) s = cap * tanhf(s / cap);
+  if (cap > 0.f) s = sizeof(T) == 4 ? cap * tanhf(s / cap) : cap - __fdividef(2.f * cap, 1.f + __expf(fminf(__fdividef(2.f * s, cap), 80.f)));
   return s - slope * (float)back;
 }
 
@@ -212,7 +214,7 @@ __global__ void __launch_bounds__(128) ll_attn_prefill_kernel(const __grid_const
         const int c = sub * 16 + d;
         if (c < a.dkp) s += q[d] * sK[kk * a.dkp + c];
       }
-      s = ll_score(ll_group_sum<TPR>(s), a.scale, a.softcap, slope, i - p);
+      s = ll_score<T>(ll_group_sum<TPR>(s), a.scale, a.softcap, slope, i - p);
       if (!live || p > i || !(a.window <= 0 || i - p < a.window || p < a.keep)) continue;
       const float mn = fmaxf(m, s);
       const float corr = expf(m - mn), pr = expf(s - mn);
@@ -312,7 +314,7 @@ __global__ void __launch_bounds__(128) ll_attn_decode_kernel(const __grid_consta
         for (int j = 0; j < KB; ++j) s[j] += __shfl_xor_sync(0xffffffffu, s[j], d);
 #pragma unroll
       for (int j = 0; j < KB; ++j) {
-        s[j] = e0 + j < hi ? ll_score(s[j], a.scale, a.softcap, slope[x], back[j]) : -INFINITY;
+        s[j] = e0 + j < hi ? ll_score<T>(s[j], a.scale, a.softcap, slope[x], back[j]) : -INFINITY;
         mn = fmaxf(mn, s[j]);
       }
       const float c = expf(m[x] - mn);            // the first key of a group is always real, so mn is finite

@@ -110,7 +110,7 @@ __global__ void __launch_bounds__(256) ll_embed_norm_kernel(const int* __restric
       for (int e = 0; e < V; ++e) v[e] = 0.f;
     }
   };
-  ll_row_norm<TPR, V>(d, mode, w, b, eps, red, get, get, [&](int i, const float (&v)[V]) { ll_put(x + (long long)r * d + i, v); });
+  ll_row_norm<TPR, V, 8>(d, mode, w, b, eps, red, get, get, [&](int i, const float (&v)[V]) { ll_put(x + (long long)r * d + i, v); });
 }
 
 template <typename T, int TPR, int V>
@@ -149,7 +149,7 @@ __global__ void __launch_bounds__(256) ll_add_norm_kernel(const float* __restric
     }
     return;
   }
-  ll_row_norm<TPR, V>(d, mode, w, b, eps, red, get,
+  ll_row_norm<TPR, V, 8>(d, mode, w, b, eps, red, get,
                       [&](int i, float (&v)[V]) { if (x_out) ll_get(x_out + (long long)r * d + i, v); else add(i, v); },
                       [&](int i, const float (&v)[V]) { ll_put(out + r * ldo + i, v); });
   for (int i = d + threadIdx.x % TPR; i < ldo; i += TPR) out[r * ldo + i] = Cvt<T>::from_f(0.f);

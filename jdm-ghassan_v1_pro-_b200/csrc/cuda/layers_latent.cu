@@ -25,22 +25,26 @@ __device__ __forceinline__ void ll_latent_row(const gb_ll_latent_args& a, int r)
   const T* src = reinterpret_cast<const T*>(a.proj) + r * a.ld_proj + a.q_rank;
   T* dst = reinterpret_cast<T*>(a.cache) + ((long long)b * a.cap + pos) * a.ldc;
   auto get = [&](int i, float (&v)[V]) { ll_get(src + i, v); };
-  ll_row_norm<32, V>(a.rank, GB_LL_NORM_RMS, a.kv_norm, nullptr, a.eps, nullptr, get, get, [&](int i, const float (&v)[V]) { ll_put(dst + i, v); });
+  ll_row_norm<32, V, 4>(a.rank, GB_LL_NORM_RMS, a.kv_norm, nullptr, a.eps, nullptr, get, get, [&](int i, const float (&v)[V]) { ll_put(dst + i, v); });
   const float2* cs = reinterpret_cast<const float2*>(a.cs) + (long long)r * (a.rot_dims / 2);
   for (int e = lane; e < a.ldc - a.rank; e += 32)
     dst[a.rank + e] = Cvt<T>::from_f(e < a.dr ? ll_turned(src + a.rank, e, a.rot_dims, cs) : 0.f);
 }
 
+// Two warps per row: one for the latent and the rotated part, one for the query latent.
 template <typename T, int V>
 __global__ void __launch_bounds__(256) ll_latent_store_kernel(const __grid_constant__ gb_ll_latent_args a) {
   pdl_wait();
-  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int w = blockIdx.x * 8 + (threadIdx.x >> 5), r = w >> 1, lane = threadIdx.x & 31;
   if (r >= a.B * a.n) return;
-  ll_latent_row<T, V>(a, r);
+  if (w & 1) {
+    ll_latent_row<T, V>(a, r);
+    return;
+  }
   const T* src = reinterpret_cast<const T*>(a.proj) + r * a.ld_proj;
   T* dst = reinterpret_cast<T*>(a.cq) + r * a.ld_cq;
   auto get = [&](int i, float (&v)[V]) { ll_get(src + i, v); };
-  ll_row_norm<32, V>(a.q_rank, GB_LL_NORM_RMS, a.q_norm, nullptr, a.eps, nullptr, get, get, [&](int i, const float (&v)[V]) { ll_put(dst + i, v); });
+  ll_row_norm<32, V, 4>(a.q_rank, GB_LL_NORM_RMS, a.q_norm, nullptr, a.eps, nullptr, get, get, [&](int i, const float (&v)[V]) { ll_put(dst + i, v); });
   for (int i = a.q_rank + lane; i < a.ld_cq; i += 32) dst[i] = Cvt<T>::from_f(0.f);
 }
 
@@ -85,72 +89,89 @@ __global__ void __launch_bounds__(256) ll_latent_queries_kernel(const __grid_con
     dst[e] = e < a.dn ? src[e] : Cvt<T>::from_f(e < dk ? ll_turned(src + a.dn, e - a.dn, a.rot_dims, cs) : 0.f);
 }
 
-// grid (row groups, H [+ 1]): qa[r, h, :] = (key map of h)^T applied to the unrotated query, then its rotated part.  Eight warps
-// share the sum over the query's dimensions.  Block row H, when there is one, writes the cache rows.
+// grid (row groups, H [+ 1], runs of 256 columns): qa[r, h, :] = (key map of h)^T applied to the unrotated query, then its rotated
+// part.  Eight warps share the sum over the query's dimensions; the first pieces of the map are requested before the wait for
+// the kernel ahead.  Block row H, when there is one, writes the cache rows.
 template <typename T, int V, int RB>
 __global__ void __launch_bounds__(256) ll_latent_absorb_kernel(const __grid_constant__ gb_ll_latent_args a) {
   __shared__ float sq[RB][256];
-  __shared__ float part[8][256];
+  __shared__ __align__(16) float part[8][256];
+  constexpr int PF = sizeof(T) == 4 ? 4 : 8;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, r0 = blockIdx.x * RB, nr = min(RB, a.B * a.n - r0), dk = a.dn + a.dr;
-  pdl_wait();
+  const int c0 = blockIdx.z * 256, c = c0 + lane * 8;
   if (h == a.H) {
-    for (int k = warp; k < nr; k += 8) ll_latent_row<T, V>(a, r0 + k);
+    pdl_wait();
+    if (blockIdx.z == 0)
+      for (int k = warp; k < nr; k += 8) ll_latent_row<T, V>(a, r0 + k);
     return;
   }
+  const T* W = reinterpret_cast<const T*>(a.W_kv) + (long long)h * a.dkp * a.ld_w + c;
+  LlRaw8<T> raw[PF];
+#pragma unroll
+  for (int i = 0; i < PF; ++i)
+    if (c < a.rank && warp + 8 * i < a.dn) raw[i].load(W + (long long)(warp + 8 * i) * a.ld_w);
+  pdl_wait();
+  auto put = [&](int k, int col, float v) {
+    const long long r = r0 + k;
+    if (a.qa16) reinterpret_cast<T*>(a.qa16)[(r * a.heads_pad + h) * a.ld_qa16 + col] = Cvt<T>::from_f(v);
+    else a.qa[(r * a.H + h) * a.ldc + col] = v;
+  };
   for (int x = threadIdx.x; x < nr * dk; x += 256) {
     const int k = x / dk, e = x - k * dk, r = r0 + k;
     const T* src = reinterpret_cast<const T*>(a.qc) + r * a.ld_qc + (long long)h * dk;
     const float2* cs = reinterpret_cast<const float2*>(a.cs) + (long long)r * (a.rot_dims / 2);
     const float v = e < a.dn ? Cvt<T>::to_f(src[e]) : ll_turned(src + a.dn, e - a.dn, a.rot_dims, cs);
     sq[k][e] = v;
-    if (e >= a.dn) a.qa[((long long)r * a.H + h) * a.ldc + a.rank + e - a.dn] = v;
+    if (e >= a.dn && blockIdx.z == 0) put(k, a.rank + e - a.dn, v);
   }
   __syncthreads();
-  const T* W = reinterpret_cast<const T*>(a.W_kv) + (long long)h * a.dkp * a.ld_w;
-  for (int c0 = 0; c0 < a.rank; c0 += 256) {
-    const int c = c0 + lane * 8;
-    float acc[RB][8];
+  float acc[RB][8];
 #pragma unroll
-    for (int k = 0; k < RB; ++k)
+  for (int k = 0; k < RB; ++k)
 #pragma unroll
-      for (int e = 0; e < 8; ++e) acc[k][e] = 0.f;
-    if (c < a.rank) {
-#pragma unroll 4
-      for (int d = warp; d < a.dn; d += 8) {
-        float w[8];
-        ll_load8(W + (long long)d * a.ld_w + c, w);
-#pragma unroll
-        for (int k = 0; k < RB; ++k) {
-          const float q = sq[k][d];
-#pragma unroll
-          for (int e = 0; e < 8; ++e) acc[k][e] += q * w[e];
-        }
-      }
-    }
+    for (int e = 0; e < 8; ++e) acc[k][e] = 0.f;
+  auto add = [&](int d, const LlRaw8<T>& x) {
+    float w[8];
+    x.expand(w);
 #pragma unroll
     for (int k = 0; k < RB; ++k) {
-      if (k >= nr) break;
-      __syncthreads();
+      const float q = sq[k][d];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) part[warp][e * 32 + lane] = acc[k][e];
-      __syncthreads();
-      const int e = threadIdx.x >> 5, col = c0 + lane * 8 + e;
-      float s = 0.f;
-#pragma unroll
-      for (int w = 0; w < 8; ++w) s += part[w][threadIdx.x];
-      if (col < a.rank) a.qa[((long long)(r0 + k) * a.H + h) * a.ldc + col] = s;
+      for (int e = 0; e < 8; ++e) acc[k][e] += q * w[e];
     }
+  };
+  if (c < a.rank) {
+#pragma unroll
+    for (int i = 0; i < PF; ++i)
+      if (warp + 8 * i < a.dn) add(warp + 8 * i, raw[i]);
+#pragma unroll 4
+    for (int d = warp + 8 * PF; d < a.dn; d += 8) {
+      LlRaw8<T> x;
+      x.load(W + (long long)d * a.ld_w);
+      add(d, x);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < RB; ++k) {
+    if (k >= nr) break;
+    if (k > 0) __syncthreads();
+    ll_store8(&part[warp][8 * lane], acc[k]);
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) s += part[w][threadIdx.x];
+    if (c0 + threadIdx.x < a.rank) put(k, c0 + threadIdx.x, s);
   }
 }
 
-// grid (rows * ceil(H / GQ), splits), 4 warps, GQ heads per block.  Lane l holds the pairs 2 (l + 32 k) of a stored row; each
-// warp walks its keys with an online soft-max per head.
 template <typename T>
 __device__ __forceinline__ float2 ll_pair(const T* p) {
   if constexpr (sizeof(T) == 4) return *reinterpret_cast<const float2*>(p);
   else return Cvt<T>::unpack2(*reinterpret_cast<const uint32_t*>(p));
 }
 
+// grid (rows * ceil(H / GQ), splits), 4 warps, GQ heads per block.  Lane l holds the pairs 2 (l + 32 k) of a stored row; each
+// warp walks its keys with an online soft-max per head.
 template <typename T, int NV, int GQ>
 __global__ void __launch_bounds__(128) ll_latent_attn_kernel(const __grid_constant__ gb_ll_latent_args a) {
   pdl_wait();
@@ -239,30 +260,51 @@ __global__ void __launch_bounds__(128) ll_latent_attn_kernel(const __grid_consta
       f[w] = sm_m[w][x] == -INFINITY ? 0.f : expf(sm_m[w][x] - mm);
       ll += sm_l[w][x] * f[w];
     }
-    float* dst = a.scratch + (((long long)r * a.H + h0 + x) * a.splits + split) * (a.ldc + 2);
-    if (threadIdx.x == 0) { dst[0] = mm; dst[1] = ll; }
+    const long long at = ((long long)r * a.H + h0 + x) * a.splits + split;
+    float* dst = a.scratch + at * a.ldc;
+    if (threadIdx.x == 0) {
+      float* ml = a.scratch + (long long)a.B * a.n * a.H * a.splits * a.ldc + 2 * at;
+      ml[0] = mm;
+      ml[1] = ll;
+    }
     for (int c = threadIdx.x; c < a.rank; c += 128) {
       const float* so = reinterpret_cast<const float*>(sm_o);
       float v = 0.f;
 #pragma unroll
       for (int w = 0; w < 4; ++w) v += so[w * W + c] * f[w];
-      dst[2 + c] = v;
+      dst[c] = v;
     }
   }
 }
 
-// One block per (row, head): the splits' results, the head's value map, the output gate.
+// One block per (row, head): the splits' results, the head's value map, the output gate.  Groups of threads take every g-th
+// split; the value map is on its way to the L2 cache before the wait for the kernel ahead.
+constexpr int LM_THREADS = 512;
 template <typename T>
-__global__ void __launch_bounds__(256) ll_latent_merge_kernel(const __grid_constant__ gb_ll_latent_args a) {
+__global__ void __launch_bounds__(LM_THREADS) ll_latent_merge_kernel(const __grid_constant__ gb_ll_latent_args a) {
   __shared__ float s_f[64];
-  __shared__ float s_o[1024 + 8];
+  __shared__ __align__(16) float s_p[LM_THREADS * 4];
+  __shared__ __align__(16) float s_o[1024 + 8];
   const int r = blockIdx.x / a.H, h = blockIdx.x - r * a.H, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int stride = a.ldc + 2, units = (a.rank + 7) / 8;
-  const float* base = a.scratch + ((long long)r * a.H + h) * a.splits * stride;
+  const int units = (a.rank + 7) / 8, quads = 2 * units, ng = min(a.splits, LM_THREADS / quads), g = tid / quads, q = tid - g * quads;
+  const long long at = ((long long)r * a.H + h) * a.splits;
+  const float* base = a.scratch + at * a.ldc;
+  const float* ml = a.scratch + (long long)a.B * a.n * a.H * a.splits * a.ldc + 2 * at;
+  const T* W = reinterpret_cast<const T*>(a.W_kv) + ((long long)a.H * a.dkp + (long long)h * a.dvp) * a.ld_w;
+  {
+    const char* w8 = reinterpret_cast<const char*>(W);
+    const long long bytes = (long long)a.dv * a.ld_w * sizeof(T);
+    for (long long i = tid * 128ll; i < bytes; i += LM_THREADS * 128ll) asm volatile("prefetch.global.L2 [%0];" ::"l"(w8 + i));
+  }
   pdl_wait();
+  constexpr int AHEAD = 8;
+  float4 v[AHEAD];
+#pragma unroll
+  for (int k = 0; k < AHEAD; ++k)
+    if (g < ng && g + k * ng < a.splits) v[k] = *reinterpret_cast<const float4*>(base + (long long)(g + k * ng) * a.ldc + 4 * q);
   if (warp == 0) {
-    const float m0 = lane < a.splits ? base[lane * stride] : -INFINITY, m1 = lane + 32 < a.splits ? base[(lane + 32) * stride] : -INFINITY;
-    const float l0 = lane < a.splits ? base[lane * stride + 1] : 0.f, l1 = lane + 32 < a.splits ? base[(lane + 32) * stride + 1] : 0.f;
+    const float m0 = lane < a.splits ? ml[2 * lane] : -INFINITY, m1 = lane + 32 < a.splits ? ml[2 * lane + 64] : -INFINITY;
+    const float l0 = lane < a.splits ? ml[2 * lane + 1] : 0.f, l1 = lane + 32 < a.splits ? ml[2 * lane + 65] : 0.f;
     const float mm = warp_max(fmaxf(m0, m1));
     const float f0 = m0 == -INFINITY ? 0.f : expf(m0 - mm), f1 = m1 == -INFINITY ? 0.f : expf(m1 - mm);
     const float l = warp_sum(l0 * f0 + l1 * f1), inv = l > 0.f ? 1.f / l : 0.f;
@@ -270,20 +312,31 @@ __global__ void __launch_bounds__(256) ll_latent_merge_kernel(const __grid_const
     s_f[lane + 32] = f1 * inv;
   }
   __syncthreads();
-  for (int c = tid; c < units * 8; c += 256) {
-    float o = 0.f;
-    if (c < a.rank) {
+  if (g < ng) {
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    auto add = [&](int s, const float4& x) {
+      const float f = s_f[s];
+      if (f != 0.f) { o.x += x.x * f; o.y += x.y * f; o.z += x.z * f; o.w += x.w * f; }      // an empty split left nothing to read
+    };
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k)
+      if (g + k * ng < a.splits) add(g + k * ng, v[k]);
 #pragma unroll 4
-      for (int s = 0; s < a.splits; ++s) o += base[s * stride + 2 + c] * s_f[s];
-    }
+    for (int s = g + AHEAD * ng; s < a.splits; s += ng) add(s, *reinterpret_cast<const float4*>(base + (long long)s * a.ldc + 4 * q));
+    *reinterpret_cast<float4*>(&s_p[(g * quads + q) * 4]) = o;
+  }
+  __syncthreads();
+  for (int c = tid; c < units * 8; c += LM_THREADS) {
+    float o = 0.f;
+    if (c < a.rank)
+      for (int k = 0; k < ng; ++k) o += s_p[k * quads * 4 + c];
     s_o[c] = o;
   }
   __syncthreads();
-  const T* W = reinterpret_cast<const T*>(a.W_kv) + ((long long)a.H * a.dkp + (long long)h * a.dvp) * a.ld_w;
   const T* gate = a.gate ? reinterpret_cast<const T*>(a.gate) + r * a.ld_gate + (long long)h * a.dv : nullptr;
   T* out = reinterpret_cast<T*>(a.out) + r * a.ldo + (long long)h * a.dv;
-#pragma unroll 2
-  for (int e = warp; e < a.dv; e += 8) {
+#pragma unroll 4
+  for (int e = warp; e < a.dv; e += LM_THREADS / 32) {
     float s = 0.f;
     for (int u = lane; u < units; u += 32) {
       float w[8];
@@ -299,6 +352,11 @@ __global__ void __launch_bounds__(256) ll_latent_merge_kernel(const __grid_const
 template <typename T>
 static int ll_latent_attn_go(const gb_ll_latent_args& a, cudaStream_t st) {
   const int rows = a.B * a.n, D = a.ldc;
+  if (a.qa16) {
+    if (const int rc = gb_ll_latent_tc(&a, st)) return rc;
+    GB_PDL_LAUNCH(ll_latent_merge_kernel<T>, dim3(rows * a.H), dim3(LM_THREADS), st, a);
+    return gb_launch_rc();
+  }
 #define GO(NV, GQ) GB_PDL_LAUNCH((ll_latent_attn_kernel<T, NV, GQ>), dim3(rows * ((a.H + GQ - 1) / GQ), a.splits), dim3(128), st, a)
   if (D <= 128) GO(2, 4);
   else if (D <= 192) GO(3, 4);
@@ -306,7 +364,7 @@ static int ll_latent_attn_go(const gb_ll_latent_args& a, cudaStream_t st) {
   else if (D <= 576) GO(9, 2);
   else GO(16, 1);
 #undef GO
-  GB_PDL_LAUNCH(ll_latent_merge_kernel<T>, dim3(rows * a.H), dim3(256), st, a);
+  GB_PDL_LAUNCH(ll_latent_merge_kernel<T>, dim3(rows * a.H), dim3(LM_THREADS), st, a);
   return gb_launch_rc();
 }
 
@@ -334,7 +392,7 @@ static bool ll_latent_vec(const gb_ll_latent_args* p) {
 extern "C" int gb_ll_latent_store(const gb_ll_latent_args* p, cudaStream_t st) {
   if (const int rc = ll_latent_check(p)) return rc;
   if (!p->proj || !p->cq || !p->q_norm || !p->kv_norm || p->ld_cq < p->q_rank) return -1;
-  const dim3 grid((p->B * p->n + 7) / 8);
+  const dim3 grid((p->B * p->n + 3) / 4);
   const bool vec = ll_latent_vec(p);
 #define LS(T, V) GB_PDL_LAUNCH((ll_latent_store_kernel<T, V>), grid, dim3(256), st, *p)
   if (p->dtype == 1) { if (vec) LS(__nv_bfloat16, 8); else LS(__nv_bfloat16, 1); }
@@ -364,10 +422,10 @@ extern "C" int gb_ll_latent_queries(const gb_ll_latent_args* p, cudaStream_t st)
 
 extern "C" int gb_ll_latent_absorb(const gb_ll_latent_args* p, int store, cudaStream_t st) {
   if (const int rc = ll_latent_check(p)) return rc;
-  if (!p->qc || !p->qa || !p->W_kv || (store && (!p->proj || !p->kv_norm))) return -1;
+  if (!p->qc || (!p->qa && !p->qa16) || !p->W_kv || (p->qa16 && p->dtype != 1) || (store && (!p->proj || !p->kv_norm))) return -1;
   const int rows = p->B * p->n, rb = rows > 1 ? 4 : 1;
   const bool vec = ll_latent_vec(p);
-  const dim3 grid((rows + rb - 1) / rb, p->H + (store ? 1 : 0));
+  const dim3 grid((rows + rb - 1) / rb, p->H + (store ? 1 : 0), (p->rank + 255) / 256);
 #define LA(T, V) do { if (rb == 1) GB_PDL_LAUNCH((ll_latent_absorb_kernel<T, V, 1>), grid, dim3(256), st, *p); \
                       else GB_PDL_LAUNCH((ll_latent_absorb_kernel<T, V, 4>), grid, dim3(256), st, *p); } while (0)
   if (p->dtype == 1) { if (vec) LA(__nv_bfloat16, 8); else LA(__nv_bfloat16, 1); }
@@ -378,6 +436,6 @@ extern "C" int gb_ll_latent_absorb(const gb_ll_latent_args* p, int store, cudaSt
 
 extern "C" int gb_ll_latent_attn(const gb_ll_latent_args* p, cudaStream_t st) {
   if (const int rc = ll_latent_check(p)) return rc;
-  if (!p->qa || !p->W_kv || !p->out || !p->scratch || p->splits < 1 || p->splits > 64) return -1;
+  if ((!p->qa && !p->qa16) || (p->qa16 && p->dtype != 1) || !p->W_kv || !p->out || !p->scratch || p->splits < 1 || p->splits > 64) return -1;
   return p->dtype == 1 ? ll_latent_attn_go<__nv_bfloat16>(*p, st) : ll_latent_attn_go<float>(*p, st);
 }

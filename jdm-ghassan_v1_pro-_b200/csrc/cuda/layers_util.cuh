@@ -39,6 +39,27 @@ __device__ __forceinline__ void ll_store8(float* p, const float (&v)[8]) {
   reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
   reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
 }
+// eight consecutive values as stored
+template <typename T> struct LlRaw8;
+template <> struct LlRaw8<__nv_bfloat16> {
+  uint4 q;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { q = __ldg(reinterpret_cast<const uint4*>(p)); }
+  __device__ __forceinline__ void expand(float (&v)[8]) const {
+    const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { const float2 f = Cvt<__nv_bfloat16>::unpack2(w[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
+  }
+};
+template <> struct LlRaw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) {
+    a = __ldg(reinterpret_cast<const float4*>(p));
+    b = __ldg(reinterpret_cast<const float4*>(p) + 1);
+  }
+  __device__ __forceinline__ void expand(float (&v)[8]) const {
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+};
 // log(1 + e^z), without overflow for large z
 __device__ __forceinline__ float ll_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
@@ -100,11 +121,10 @@ __device__ __forceinline__ float ll_row_sum(float v, float* red) {
 
 // Norm of one row by TPR threads, V neighbouring values at a time.  `get(i, v)` gives the values at i .. i + V - 1 and is
 // called once per place, except for places past the ones kept in registers, which `again(i, v)` gives once more; `put(i, v)`
-// takes the normed values.
-template <int TPR, int V, typename Get, typename Again, typename Put>
+// takes the normed values.  KEEP * V values per thread stay in registers.
+template <int TPR, int V, int KEEP, typename Get, typename Again, typename Put>
 __device__ __forceinline__ void ll_row_norm(int d, int mode, const float* __restrict__ w, const float* __restrict__ b, float eps, float* red,
                                             Get get, Again again, Put put) {
-  constexpr int KEEP = 8;
   const int t = threadIdx.x % TPR;
   float keep[KEEP][V];
   float sum = 0.f, dev = 0.f;

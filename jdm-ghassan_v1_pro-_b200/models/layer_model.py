@@ -275,9 +275,15 @@ class LayerModel:
         out = self.mixed(i)
         a.out, a.ldo = out.data_ptr(), out.stride(0)
         if n <= LATENT_FEW:
-            a.qa = self.buf("qa%d" % rows, m.heads * a.ldc, torch.float32, rows=rows).data_ptr()
-            blocks = rows * ((m.heads + 3) // 4)
-            a.splits = int(max(1, min(64, (592 + blocks - 1) // blocks, (cache.cap + 15) // 16)))
+            plan = K.latent_tc_plan(a) if self.use_tc else None
+            if plan is not None:
+                a.heads_pad, a.ld_qa16 = plan
+                a.qa16 = self.buf("qa16:%dx%d+%d" % (rows, m.heads, m.kv_rank + m.rot_dim), a.heads_pad * a.ld_qa16, rows=rows).data_ptr()
+                a.splits = int(max(1, min(64, 148 // (rows * ((m.heads + 31) // 32)), cache.cap // 128)))
+            else:
+                a.qa = self.buf("qa%d" % rows, m.heads * a.ldc, torch.float32, rows=rows).data_ptr()
+                blocks = rows * ((m.heads + 3) // 4)
+                a.splits = int(max(1, min(64, (592 + blocks - 1) // blocks, (cache.cap + 15) // 16)))
             a.scratch = self.buf("latent_scratch%d" % rows, m.heads * a.splits * (a.ldc + 2), torch.float32, rows=rows).data_ptr()
         else:
             a.q = self.buf("q", m.heads * a.dkp).data_ptr()

@@ -58,6 +58,7 @@ class LatentArgs(ctypes.Structure):
         ("proj", c_vp), ("ld_proj", c_ll), ("q_norm", c_vp), ("kv_norm", c_vp),
         ("cq", c_vp), ("ld_cq", c_ll), ("cache", c_vp), ("ldc", c_int), ("cap", c_int),
         ("qc", c_vp), ("ld_qc", c_ll), ("q", c_vp), ("W_kv", c_vp), ("ld_w", c_ll), ("qa", c_vp),
+        ("qa16", c_vp), ("heads_pad", c_int), ("ld_qa16", c_int),
         ("gate", c_vp), ("ld_gate", c_ll), ("out", c_vp), ("ldo", c_ll),
         ("scratch", c_vp), ("splits", c_int), ("st", c_vp), ("status", c_vp),
     ]
@@ -179,6 +180,12 @@ def latent_queries(a: LatentArgs):
 
 def latent_absorb(a: LatentArgs, store: bool):
     _call("gb_ll_latent_absorb", ctypes.byref(a), c_int(int(store)))
+
+
+def latent_tc_plan(a: LatentArgs):
+    """(heads_pad, ld_qa16) of the tensor-core kernel, or None when it does not cover the shapes."""
+    hp, ld = c_int(0), c_int(0)
+    return (hp.value, ld.value) if _lib.lib().gb_ll_latent_tc_plan(ctypes.byref(a), ctypes.byref(hp), ctypes.byref(ld)) == 0 else None
 
 
 def latent_attn(a: LatentArgs):

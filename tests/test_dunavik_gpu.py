@@ -232,14 +232,14 @@ def test_gemv_prologues(dtype, B, d, N, n1):
     near(out, (v / torch.sqrt((v * v).mean(-1, keepdim=True) + 1e-4) * w1.double()) @ W.t(), tol)
 
 
-def _one_layer(layer, width=64, dtype=F32, slots=1, rows=512, max_len=4096, seed=0):
+def _one_layer(layer, width=64, dtype=F32, slots=1, rows=512, max_len=4096, seed=0, tc=True):
     """A model of one layer and its memory, for kernels on hand-made projections."""
     from ghassan_b200.inference.layer_cache import SlotManager
     from ghassan_b200.models.layer_list import LayerListConfig
     from ghassan_b200.models.layer_model import LayerModel
     raw = D.config([layer], width, 32)
     cfg = LayerListConfig.from_json(raw)
-    m = LayerModel(cfg, D.weights(raw, seed), slots, rows, dtype)
+    m = LayerModel(cfg, D.weights(raw, seed), slots, rows, dtype, use_tensor_cores=tc)
     mem = SlotManager(cfg, slots, max_len, rows, dtype, m.dev)
     return m, mem, torch.zeros(slots, 4, dtype=torch.int32, device="cuda")
 
@@ -377,14 +377,15 @@ def test_latent_rows_and_queries(dtype, sizes, pos):
     assert float(got[..., sizes[1] + sizes[2]:].abs().sum()) == 0.0
 
 
-@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("dtype, tc", [(F32, False), (BF, False), (BF, True)], ids=["fp32", "general", "tc"])
 @pytest.mark.parametrize("sizes", LATENTS, ids=["x".join(map(str, s)) for s in LATENTS])
-@pytest.mark.parametrize("portions", [(200,), (1,) * 70, (130, 1, 2, 3, 4, 1, 59), (2, 5, 4, 140, 3)], ids=["whole", "tokens", "mixed", "few"])
-def test_latent_attention_of_portions(dtype, sizes, portions):
+@pytest.mark.parametrize("portions", [(200,), (1,) * 70, (130, 1, 2, 3, 4, 1, 59), (2, 5, 4, 140, 3), (505, 1, 1, 1, 3)],
+                         ids=["whole", "tokens", "mixed", "few", "long"])
+def test_latent_attention_of_portions(dtype, tc, sizes, portions):
     """Keys and values made for a pass, and queries against the latents themselves, over one cache."""
     from ghassan_b200.ops import _lib
     from ghassan_b200.ops import layers as K
-    m, mem, state = _one_layer(D.latent(*sizes), dtype=dtype)
+    m, mem, state = _one_layer(D.latent(*sizes), dtype=dtype, tc=tc)
     T, w = sum(portions), m.weights[0]
     proj = _projection(m, T)
     want = _latent_reference(m, proj, range(T), dtype)[3]
@@ -403,6 +404,40 @@ def test_latent_attention_of_portions(dtype, sizes, portions):
         lo += n
     _lib.check_status(m.dev)
     near(torch.cat(got), want, 2e-5 if dtype == F32 else 2.0 ** -5)
+
+
+@pytest.mark.parametrize("H, rank, dr", [(5, 96, 32), (16, 256, 64), (20, 512, 64), (40, 64, 16), (33, 640, 64)])
+@pytest.mark.parametrize("splits", [1, 2, 5])
+def test_latent_tensor_core_partials(H, rank, dr, splits):
+    """Runs of several tiles with a growing maximum, one key far above the others, against the plain soft-max; rows of the cache
+    past the sequence hold other numbers."""
+    from ghassan_b200.ops import _lib
+    from ghassan_b200.ops import layers as K
+    m, mem, state = _one_layer(D.latent(H, 16, dr, 24, rank, 32), dtype=BF, max_len=1500)
+    g = torch.Generator().manual_seed(H)
+    count = 1203
+    c = mem.layers[0]
+    c.rows[0, :, :rank + dr] = torch.randn(c.cap, rank + dr, generator=g).to(BF).cuda()
+    c.rows[0, :count] *= torch.linspace(0.3, 1.0, count, device="cuda").to(BF)[:, None]
+    state[:, 0] = count - 1
+    m._rotations(state, 1, 1)
+    a = m.latent_args(0, c, state, 0, 1, 1)
+    a.scale, a.splits = 0.1, splits
+    scratch = torch.zeros(H * splits * (a.ldc + 2), device="cuda")
+    a.scratch = scratch.data_ptr()
+    qa = torch.zeros(a.heads_pad, a.ld_qa16, dtype=BF, device="cuda")
+    qa[:H, :rank + dr] = torch.randn(H, rank + dr, generator=g).to(BF).cuda() * (10.0 * (rank + dr) ** -0.5)
+    qa[1, :rank + dr] = c.rows[0, 131, :rank + dr] * 0.6
+    a.qa16 = qa.data_ptr()
+    gate = torch.full((1, H * 24), 50.0, dtype=BF, device="cuda")
+    a.gate, a.ld_gate = gate.data_ptr(), H * 24
+    K.latent_attn(a)
+    _lib.check_status(m.dev)
+    rows = c.rows[0, :count, :rank + dr].double().cpu().numpy()
+    s = qa[:H, :rank + dr].double().cpu().numpy() @ rows.T * 0.1
+    o = O.softmax(s, np.ones_like(s, dtype=bool)) @ rows[:, :rank]
+    values = m.weights[0].w_kv[H * a.dkp:].view(H, a.dvp, -1)[:, :24, :rank].double().cpu().numpy()
+    near(m.mixed(0)[:1, :H * 24].view(H, 24), np.einsum("hvr,hr->hv", values, o), 2.0 ** -6)
 
 
 # ------------------------------------------------------------------------------------------------ long decoding, slots, batches

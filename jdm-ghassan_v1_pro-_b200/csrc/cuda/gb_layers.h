@@ -100,7 +100,8 @@ typedef struct gb_ll_attn_args {
   void* cache_k; void* cache_v;          // [B, cap, ld_k]: head g at column g*dkp / [B, cap, ld_v]: at g*dvp
   long long ld_k, ld_v;
   void* out; long long ldo;              // [rows, H*dv]
-  float* scratch; int splits;            // token step: B * H * splits * (dvp + 2) floats
+  float* scratch; int splits;            // token step: B * H * splits * (dvp + 2) floats: partial outputs,
+                                         // then (maximum, sum) pairs
   const gb_seq_state* st;
   int pos0_max;                          // host's upper bound of abs_pos over the B sequences (tile counts); -1 unknown
   int* status;

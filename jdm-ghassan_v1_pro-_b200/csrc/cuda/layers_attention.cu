@@ -351,45 +351,67 @@ __global__ void __launch_bounds__(128) ll_attn_decode_kernel(const __grid_consta
       ll += sm_l[w][x] * f;
       oo += sm_o[w][x][c] * f;
     }
-    float* dst = a.scratch + (((long long)b * a.H + h0 + x) * a.splits + split) * (a.dvp + 2);
-    dst[2 + c] = oo;
-    if (c == 0) { dst[0] = mm; dst[1] = ll; }
+    const long long at = ((long long)b * a.H + h0 + x) * a.splits + split;
+    a.scratch[at * a.dvp + c] = oo;
+    if (c == 0) *reinterpret_cast<float2*>(a.scratch + (long long)a.B * a.H * a.splits * a.dvp + 2 * at) = make_float2(mm, ll);
   }
 }
 
-// One block per (sequence, head): the splits' results, the sink and the output gate.
+// One block per (sequence, head): the splits' results, the sink and the output gate.  Groups of threads take every g-th split.
 template <typename T>
-__global__ void __launch_bounds__(128) ll_attn_merge_kernel(const __grid_constant__ gb_ll_attn_args a) {
+__global__ void __launch_bounds__(256) ll_attn_merge_kernel(const __grid_constant__ gb_ll_attn_args a) {
   pdl_wait();
   __shared__ float s_f[128];
   __shared__ float s_red[8];
+  __shared__ __align__(16) float s_p[256 * 4];
   const int b = blockIdx.x / a.H, h = blockIdx.x - b * a.H, tid = threadIdx.x;
-  const int stride = a.dvp + 2;
-  const float* base = a.scratch + ((long long)b * a.H + h) * a.splits * stride;
-  const float ms = tid < a.splits ? base[tid * stride] : -INFINITY;
-  const float ls = tid < a.splits ? base[tid * stride + 1] : 0.f;
-  float mm = warp_max(ms);
-  if ((tid & 31) == 0) s_red[tid >> 5] = mm;
+  const int quads = a.dvp / 4, ng = min(a.splits, 256 / quads), g = tid / quads, q = tid - g * quads;
+  const long long at = ((long long)b * a.H + h) * a.splits;
+  const float* base = a.scratch + at * a.dvp + 4 * q;
+  const float2* ml = reinterpret_cast<const float2*>(a.scratch + (long long)a.B * a.H * a.splits * a.dvp + 2 * at);
+  constexpr int AHEAD = 4;
+  float4 v[AHEAD];
+#pragma unroll
+  for (int k = 0; k < AHEAD; ++k)
+    if (g < ng && g + k * ng < a.splits) v[k] = *reinterpret_cast<const float4*>(base + (long long)(g + k * ng) * a.dvp);
+  const float2 own = tid < a.splits ? ml[tid] : make_float2(-INFINITY, 0.f);       // up to 128 splits: the first four warps
+  float mm = warp_max(own.x);
+  if ((tid & 31) == 0 && tid < 128) s_red[tid >> 5] = mm;
   __syncthreads();
   mm = fmaxf(fmaxf(s_red[0], s_red[1]), fmaxf(s_red[2], s_red[3]));
   if (a.sink) mm = fmaxf(mm, a.sink[h]);
-  const float f = ms == -INFINITY ? 0.f : expf(ms - mm);
-  s_f[tid] = f;
-  const float lw = warp_sum(ls * f);
-  if ((tid & 31) == 0) s_red[4 + (tid >> 5)] = lw;
+  const float f = own.x == -INFINITY ? 0.f : expf(own.x - mm);
+  const float lw = warp_sum(own.y * f);
+  if (tid < 128) {
+    s_f[tid] = f;
+    if ((tid & 31) == 0) s_red[4 + (tid >> 5)] = lw;
+  }
   __syncthreads();
   float l = s_red[4] + s_red[5] + s_red[6] + s_red[7];
   if (a.sink) l += expf(a.sink[h] - mm);
   const float inv = l > 0.f ? 1.f / l : 0.f;
+  if (g < ng) {
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    auto add = [&](int s, const float4& x) {
+      const float w = s_f[s];
+      o.x += x.x * w; o.y += x.y * w; o.z += x.z * w; o.w += x.w * w;
+    };
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k)
+      if (g + k * ng < a.splits) add(g + k * ng, v[k]);
+#pragma unroll 4
+    for (int s = g + AHEAD * ng; s < a.splits; s += ng) add(s, *reinterpret_cast<const float4*>(base + (long long)s * a.dvp));
+    *reinterpret_cast<float4*>(&s_p[tid * 4]) = o;
+  }
+  __syncthreads();
   const T* gate = reinterpret_cast<const T*>(a.gate) + b * a.ld_gate + h * a.dv;
   T* op = reinterpret_cast<T*>(a.out) + b * a.ldo + h * a.dv;
-  for (int c = tid; c < a.dv; c += 128) {
+  for (int c = tid; c < a.dv; c += 256) {
     float o = 0.f;
-#pragma unroll 8
-    for (int s = 0; s < a.splits; ++s) o += base[s * stride + 2 + c] * s_f[s];
-    float v = o * inv;
-    if (a.gate) v *= ll_sigmoid(Cvt<T>::to_f(gate[c]));
-    op[c] = Cvt<T>::from_f(v);
+    for (int k = 0; k < ng; ++k) o += s_p[k * a.dvp + c];
+    float v1 = o * inv;
+    if (a.gate) v1 *= ll_sigmoid(Cvt<T>::to_f(gate[c]));
+    op[c] = Cvt<T>::from_f(v1);
   }
 }
 
@@ -401,7 +423,7 @@ static void ll_decode_go(const gb_ll_attn_args& a, cudaStream_t st) {
   else if (R == 2) GO(2);
   else GO(4);
 #undef GO
-  GB_PDL_LAUNCH(ll_attn_merge_kernel<T>, dim3(a.B * a.H), dim3(128), st, a);
+  GB_PDL_LAUNCH(ll_attn_merge_kernel<T>, dim3(a.B * a.H), dim3(256), st, a);
 }
 
 template <typename T>

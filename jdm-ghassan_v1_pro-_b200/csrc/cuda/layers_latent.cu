@@ -277,31 +277,38 @@ __global__ void __launch_bounds__(128) ll_latent_attn_kernel(const __grid_consta
   }
 }
 
-// One block per (row, head): the splits' results, the head's value map, the output gate.  Groups of threads take every g-th
-// split; the value map is on its way to the L2 cache before the wait for the kernel ahead.
-constexpr int LM_THREADS = 512;
+// A cluster of four blocks per (row, head): the splits' results, the head's value map, the output gate.  Each block combines a
+// quarter of the latent dimensions (groups of threads take every g-th split), gives them to all four, and makes a quarter of
+// the head's outputs; its first rows of the value map are requested before the wait for the kernel ahead.
+constexpr int LM_THREADS = 512, LM_CL = 4;
 template <typename T>
-__global__ void __launch_bounds__(LM_THREADS) ll_latent_merge_kernel(const __grid_constant__ gb_ll_latent_args a) {
+__global__ void __cluster_dims__(LM_CL, 1, 1) __launch_bounds__(LM_THREADS) ll_latent_merge_kernel(const __grid_constant__ gb_ll_latent_args a) {
   __shared__ float s_f[64];
   __shared__ __align__(16) float s_p[LM_THREADS * 4];
-  __shared__ __align__(16) float s_o[1024 + 8];
-  const int r = blockIdx.x / a.H, h = blockIdx.x - r * a.H, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int units = (a.rank + 7) / 8, quads = 2 * units, ng = min(a.splits, LM_THREADS / quads), g = tid / quads, q = tid - g * quads;
+  __shared__ __align__(16) float s_o[1024];
+  constexpr int WARPS = LM_THREADS / 32;
+  const int item = blockIdx.x / LM_CL, rank = blockIdx.x % LM_CL, r = item / a.H, h = item - r * a.H, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int units = (a.rank + 7) / 8, mine = (2 * units + LM_CL - 1) / LM_CL;         // quads of dimensions per block
+  const int ng = min(a.splits, LM_THREADS / mine), g = tid / mine, q = rank * mine + tid - g * mine;
+  const bool works = g < ng && q < 2 * units;
   const long long at = ((long long)r * a.H + h) * a.splits;
-  const float* base = a.scratch + at * a.ldc;
+  const float* base = a.scratch + at * a.ldc + 4 * q;
   const float* ml = a.scratch + (long long)a.B * a.n * a.H * a.splits * a.ldc + 2 * at;
   const T* W = reinterpret_cast<const T*>(a.W_kv) + ((long long)a.H * a.dkp + (long long)h * a.dvp) * a.ld_w;
-  {
-    const char* w8 = reinterpret_cast<const char*>(W);
-    const long long bytes = (long long)a.dv * a.ld_w * sizeof(T);
-    for (long long i = tid * 128ll; i < bytes; i += LM_THREADS * 128ll) asm volatile("prefetch.global.L2 [%0];" ::"l"(w8 + i));
-  }
+  const int per = (a.dv + LM_CL - 1) / LM_CL, e_lo = rank * per + warp, e_hi = min(a.dv, (rank + 1) * per);
+  constexpr int PW = 2;                                      // rows and pieces of 256 columns that are requested ahead
+  LlRaw8<T> raw[PW][PW];
+#pragma unroll
+  for (int i = 0; i < PW; ++i)
+#pragma unroll
+    for (int k = 0; k < PW; ++k)
+      if (e_lo + i * WARPS < e_hi && lane + 32 * k < units) raw[i][k].load(W + (long long)(e_lo + i * WARPS) * a.ld_w + (lane + 32 * k) * 8);
   pdl_wait();
-  constexpr int AHEAD = 8;
+  constexpr int AHEAD = 4;
   float4 v[AHEAD];
 #pragma unroll
   for (int k = 0; k < AHEAD; ++k)
-    if (g < ng && g + k * ng < a.splits) v[k] = *reinterpret_cast<const float4*>(base + (long long)(g + k * ng) * a.ldc + 4 * q);
+    if (works && g + k * ng < a.splits) v[k] = *reinterpret_cast<const float4*>(base + (long long)(g + k * ng) * a.ldc);
   if (warp == 0) {
     const float m0 = lane < a.splits ? ml[2 * lane] : -INFINITY, m1 = lane + 32 < a.splits ? ml[2 * lane + 64] : -INFINITY;
     const float l0 = lane < a.splits ? ml[2 * lane + 1] : 0.f, l1 = lane + 32 < a.splits ? ml[2 * lane + 65] : 0.f;
@@ -311,42 +318,69 @@ __global__ void __launch_bounds__(LM_THREADS) ll_latent_merge_kernel(const __gri
     s_f[lane] = f0 * inv;
     s_f[lane + 32] = f1 * inv;
   }
-  __syncthreads();
+  cluster_sync_all();                                        // s_f is there, and the other blocks run
   if (g < ng) {
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
     auto add = [&](int s, const float4& x) {
       const float f = s_f[s];
       if (f != 0.f) { o.x += x.x * f; o.y += x.y * f; o.z += x.z * f; o.w += x.w * f; }      // an empty split left nothing to read
     };
+    if (works) {
 #pragma unroll
-    for (int k = 0; k < AHEAD; ++k)
-      if (g + k * ng < a.splits) add(g + k * ng, v[k]);
+      for (int k = 0; k < AHEAD; ++k)
+        if (g + k * ng < a.splits) add(g + k * ng, v[k]);
 #pragma unroll 4
-    for (int s = g + AHEAD * ng; s < a.splits; s += ng) add(s, *reinterpret_cast<const float4*>(base + (long long)s * a.ldc + 4 * q));
-    *reinterpret_cast<float4*>(&s_p[(g * quads + q) * 4]) = o;
+      for (int s = g + AHEAD * ng; s < a.splits; s += ng) add(s, *reinterpret_cast<const float4*>(base + (long long)s * a.ldc));
+    }
+    *reinterpret_cast<float4*>(&s_p[tid * 4]) = o;
   }
   __syncthreads();
-  for (int c = tid; c < units * 8; c += LM_THREADS) {
+  for (int c = tid; c < 4 * mine; c += LM_THREADS) {
+    const int dim = rank * 4 * mine + c;
+    if (dim >= units * 8) break;
     float o = 0.f;
-    if (c < a.rank)
-      for (int k = 0; k < ng; ++k) o += s_p[k * quads * 4 + c];
-    s_o[c] = o;
+    if (dim < a.rank)
+      for (int k = 0; k < ng; ++k) o += s_p[k * mine * 4 + c];
+#pragma unroll
+    for (int to = 0; to < LM_CL; ++to)
+      asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(mapa_shared(smem_u32(&s_o[dim]), to)), "f"(o) : "memory");
   }
-  __syncthreads();
+  cluster_sync_all();
   const T* gate = a.gate ? reinterpret_cast<const T*>(a.gate) + r * a.ld_gate + (long long)h * a.dv : nullptr;
   T* out = reinterpret_cast<T*>(a.out) + r * a.ldo + (long long)h * a.dv;
-#pragma unroll 4
-  for (int e = warp; e < a.dv; e += LM_THREADS / 32) {
-    float s = 0.f;
-    for (int u = lane; u < units; u += 32) {
-      float w[8];
-      ll_load8(W + (long long)e * a.ld_w + u * 8, w);
+  auto dot = [&](const LlRaw8<T>& x, int u) {
+    float w[8], o[8], s = 0.f;
+    x.expand(w);
+    ll_load8(&s_o[u * 8], o);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) s += w[k] * s_o[u * 8 + k];
-    }
+    for (int k = 0; k < 8; ++k) s += w[k] * o[k];
+    return s;
+  };
+  auto finish = [&](int e, float s) {
     s = warp_sum(s);
     if (lane == 0) out[e] = Cvt<T>::from_f(gate ? s * ll_sigmoid(Cvt<T>::to_f(gate[e])) : s);
+  };
+  auto rest = [&](int e, int u0) {
+    float s = 0.f;
+    for (int u = u0; u < units; u += 32) {
+      LlRaw8<T> x;
+      x.load(W + (long long)e * a.ld_w + u * 8);
+      s += dot(x, u);
+    }
+    return s;
+  };
+#pragma unroll
+  for (int i = 0; i < PW; ++i) {
+    const int e = e_lo + i * WARPS;
+    if (e < e_hi) {
+      float s = 0.f;
+#pragma unroll
+      for (int k = 0; k < PW; ++k)
+        if (lane + 32 * k < units) s += dot(raw[i][k], lane + 32 * k);
+      finish(e, s + rest(e, lane + 32 * PW));
+    }
   }
+  for (int e = e_lo + PW * WARPS; e < e_hi; e += WARPS) finish(e, rest(e, lane));
 }
 
 template <typename T>
@@ -354,7 +388,7 @@ static int ll_latent_attn_go(const gb_ll_latent_args& a, cudaStream_t st) {
   const int rows = a.B * a.n, D = a.ldc;
   if (a.qa16) {
     if (const int rc = gb_ll_latent_tc(&a, st)) return rc;
-    GB_PDL_LAUNCH(ll_latent_merge_kernel<T>, dim3(rows * a.H), dim3(LM_THREADS), st, a);
+    GB_PDL_LAUNCH(ll_latent_merge_kernel<T>, dim3(rows * a.H * LM_CL), dim3(LM_THREADS), st, a);
     return gb_launch_rc();
   }
 #define GO(NV, GQ) GB_PDL_LAUNCH((ll_latent_attn_kernel<T, NV, GQ>), dim3(rows * ((a.H + GQ - 1) / GQ), a.splits), dim3(128), st, a)
@@ -364,7 +398,7 @@ static int ll_latent_attn_go(const gb_ll_latent_args& a, cudaStream_t st) {
   else if (D <= 576) GO(9, 2);
   else GO(16, 1);
 #undef GO
-  GB_PDL_LAUNCH(ll_latent_merge_kernel<T>, dim3(rows * a.H), dim3(LM_THREADS), st, a);
+  GB_PDL_LAUNCH(ll_latent_merge_kernel<T>, dim3(rows * a.H * LM_CL), dim3(LM_THREADS), st, a);
   return gb_launch_rc();
 }
 

@@ -113,24 +113,30 @@ __global__ void __launch_bounds__(LT_THREADS) ll_latent_tc_kernel(const __grid_c
   } else if (warp == 5) {
     if (lane == 0 && n_t > 0) {
       const uint32_t idesc_s = make_idesc_f16(1, 0, 0, AT_N, HP), idesc_o = make_idesc_f16(1, 1, 0, 128, HP);
-      const uint32_t q0 = smem_u32(sQ), p0 = smem_u32(sP);
+      const uint64_t dq0 = make_smem_desc_sw128(smem_u32(sQ), 16, 1024), dp0 = make_smem_desc_sw128(smem_u32(sP), 16, 1024);
       bool ok = at_wait(q_full, 0, a.status, ST_TIMEOUT_FULL, abort_flag);
       for (int t = 0; t < n_t && ok; ++t) {
         const int s = t % stages, ph = (t / stages) & 1;
         if (!at_wait(&kv_full[s], ph, a.status, ST_TIMEOUT_FULL, abort_flag)) break;
         tc_fence_after();
+        // descriptors step by whole panels (start addresses count 16 bytes): one thread issues, so few instructions per product
         const uint32_t k0 = smem_u32(sK + (size_t)s * panels * KP);
-        for (int kk = 0; kk < dsteps; ++kk)
-          umma_f16(tmem_S, make_smem_desc_sw128(k0 + (kk >> 2) * KP + (kk & 3) * 32, 16, 1024),
-                   make_smem_desc_sw128(q0 + (kk >> 2) * QP + (kk & 3) * 32, 16, 1024), idesc_s, kk > 0);
+        uint64_t dk = make_smem_desc_sw128(k0, 16, 1024), dq = dq0;
+        for (int kk = 0; kk < dsteps; kk += 4, dk += KP >> 4, dq += QP >> 4) {
+          const int left = dsteps - kk;
+          umma_f16(tmem_S, dk, dq, idesc_s, kk > 0);
+          if (left > 1) umma_f16(tmem_S, dk + 2, dq + 2, idesc_s, 1);
+          if (left > 2) umma_f16(tmem_S, dk + 4, dq + 4, idesc_s, 1);
+          if (left > 3) umma_f16(tmem_S, dk + 6, dq + 6, idesc_s, 1);
+        }
         umma_commit(s_full);
         if (!at_wait(p_ready, t & 1, a.status, ST_TIMEOUT_TMEM_EMPTY, abort_flag)) break;
         tc_fence_after();
-        for (int c = 0; c < chunks; ++c)
+        uint64_t dv = make_smem_desc_sw128(k0, KP, 1024);
+        for (int c = 0; c < chunks; ++c, dv += 2 * (KP >> 4))
 #pragma unroll
           for (int kk = 0; kk < AT_N / 16; ++kk)      // A: latent dimensions along M (two panels), keys along K, 16 rows a step
-            umma_f16(tmem_O + c * HP, make_smem_desc_sw128(k0 + 2 * c * KP + kk * 2048, KP, 1024),
-                     make_smem_desc_sw128(p0 + (kk >> 2) * QP + (kk & 3) * 32, 16, 1024), idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
+            umma_f16(tmem_O + c * HP, dv + kk * (2048 >> 4), dp0 + ((kk >> 2) * QP + (kk & 3) * 32) / 16, idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
         umma_commit(&kv_empty[s]);
         umma_commit(o_full);
       }
@@ -195,12 +201,16 @@ __global__ void __launch_bounds__(LT_THREADS) ll_latent_tc_kernel(const __grid_c
           }
         tmem_st_wait();
       }
+#pragma unroll
+      for (int h = 0; h < HP; h += 4) {
+        const float4 q = *reinterpret_cast<const float4*>(&s_m[h]);
+        s[h] = lt_ex2(s[h] - q.x); s[h + 1] = lt_ex2(s[h + 1] - q.y); s[h + 2] = lt_ex2(s[h + 2] - q.z); s[h + 3] = lt_ex2(s[h + 3] - q.w);
+      }
       uint8_t* panel = sP + (key >> 6) * QP;
 #pragma unroll
       for (int h = 0; h < HP; ++h) {
-        const float e = lt_ex2(s[h] - s_m[h]);
-        lsum[h] += e;
-        *reinterpret_cast<T*>(panel + sw128_off(h, key & 63)) = Cvt<T>::from_f(e);
+        lsum[h] += s[h];
+        *reinterpret_cast<T*>(panel + sw128_off(h, key & 63)) = Cvt<T>::from_f(s[h]);
       }
       tc_fence_before();
       fence_proxy_async();
@@ -225,9 +235,11 @@ __global__ void __launch_bounds__(LT_THREADS) ll_latent_tc_kernel(const __grid_c
       lt_tmem_load<HP>(tmem_O + lane_base + c * HP, rg);
       const int dim = c * 128 + key;
       if (dim < a.rank) {
+        float* dst = a.scratch + first * a.ldc + dim;
+        const int step = a.splits * a.ldc;
 #pragma unroll
-        for (int h = 0; h < HP; ++h)
-          if (h0 + h < a.H) a.scratch[(first + (long long)h * a.splits) * a.ldc + dim] = __uint_as_float(rg[h]);
+        for (int h = 0; h < HP; ++h, dst += step)
+          if (h0 + h < a.H) *dst = __uint_as_float(rg[h]);
       }
       __syncwarp();
     }

@@ -36,9 +36,10 @@ NVCC_FLAGS = [
 ]
 # Kernels of layer-list models keep IEEE division, square roots and math functions: their fp32 mode is meant to be exact.
 PRECISE_PREFIX = "layers_"
-# Sources behind one kind of model, for a process that serves nothing else and finds no library (`ensure_layers`).
-LAYERS_PART = ("layers_", "gemm_")
-LAYERS_SO = os.path.join(HERE, "_gb200_layers.so")
+# Sources behind layer-list models, for a process that serves nothing else and finds no library (`ensure_layers`): what all of
+# them need, and what a type of mixer adds.
+LAYERS_PART = ("gemm_", "layers_common", "layers_gemv", "layers_attention", "layers_attn_tc")
+MIXER_PARTS = {"latent_attention": ("layers_latent",), "mamba2": ("layers_mamba", "layers_ssd")}
 CXX_FLAGS = ["-O2", "-std=c++20", "-fPIC", "-fvisibility=hidden", "-Wall", "-Wno-unused-function",
              "-pthread"]
 
@@ -174,17 +175,18 @@ def build_cuda(verbose=False, force=False, part=None, target=None):
     return target
 
 
-def ensure_layers() -> str:
-    """Device library for a process that only serves layer-list models: the full one when it is there and up to date,
-    else a library of just the sources they need (compiled on the first call)."""
+def ensure_layers(mixers=tuple(MIXER_PARTS)) -> str:
+    """Device library for a process that only serves layer-list models with these types of mixers: the full one when it is
+    there and up to date, else a library of just the sources they need (compiled on the first call)."""
     import fcntl
-    srcs = [s for s in _sources("cuda", ".cu") if os.path.basename(s).startswith(LAYERS_PART)] + _headers("cuda")
-    if not _newer(srcs, CUDA_SO):
+    extra = sorted(k for k in MIXER_PARTS if k in mixers)
+    part = LAYERS_PART + tuple(p for k in extra for p in MIXER_PARTS[k])
+    if not _newer(_sources("cuda", ".cu") + _headers("cuda"), CUDA_SO):
         return CUDA_SO
     os.makedirs(BUILD, exist_ok=True)
     with open(os.path.join(BUILD, ".lock"), "w") as lock:
         fcntl.flock(lock, fcntl.LOCK_EX)
-        return build_cuda(part=LAYERS_PART, target=LAYERS_SO)
+        return build_cuda(part=part, target=os.path.join(HERE, "_gb200_layers%s.so" % "".join("_" + k for k in extra)))
 
 
 def build_all(verbose=False, force=False):

@@ -57,9 +57,9 @@ def main(argv: Optional[List[str]] = None) -> int:
     a = _parser().parse_args(argv)
     from .. import build as B
     from ..ops import _lib
-    _lib.use(B.ensure_layers())
     from ..inference import model_io as IO
     m = IO.load_model(a.model)
+    _lib.use(B.ensure_layers({s.mixer.kind for s in m.cfg.layers}))
     n = max(1, a.max_tokens)
     eng = IO.build_engine(m, batch=max(1, a.slots), max_len=n, fmt={"bfloat16": "bf16", "float32": "f32"}[a.dtype])
     os.makedirs(a.out, exist_ok=True)

@@ -9,7 +9,7 @@ Two schedules of the same layers:
   stand side by side: adds their sum to the residual and leaves the norm of that).
 * :meth:`LayerModel.forward_token`: one token of a few sequences: GEMV kernels whose prologues do those row-wise steps, so
   a layer is six (attention) or five (state-space) dependent launches, captured in one CUDA graph by the engine.  Side by
-  side: five (attention) or seven (latent attention).
+  side: five (attention) or six (latent attention).
 
 Weights are stored once.  Rows that feed a product are zero-padded to eight elements; gate and up rows are interleaved in
 blocks of 64 (the layout of the fused SwiGLU epilogue); all projections that read a sublayer's input are one matrix.  Where
